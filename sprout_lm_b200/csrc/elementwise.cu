@@ -36,6 +36,66 @@ SPROUT_API int sprout_embed(const void* table, int table_dtype, const int* token
   return sprout_check_launch("embed");
 }
 
+// x[t, :] = table[token[t], :] * scale + pairs[row, :], row = (previous * mul_prev + token * mul_cur) mod buckets, and the last
+// row (number `buckets`) for a sequence's first token.  A request's previous token comes from the step's tokens or, for the
+// first token it brings, from its state slot.  The block of that token reads the slot and then leaves the request's last
+// token of the step there (nobody else touches it).
+template <typename TW>
+__global__ void embed_pairs_kernel(const TW* __restrict__ table, const TW* __restrict__ pairs, const int* __restrict__ tokens,
+                                   const int* __restrict__ positions, const int* __restrict__ seq_of_token,
+                                   const int* __restrict__ q_start, const int* __restrict__ state_slots, int* __restrict__ last_token,
+                                   int num_slots, float* __restrict__ out, int hidden, int vocab, float scale, long long mul_prev,
+                                   long long mul_cur, int buckets, int* status) {
+  __shared__ int s_token, s_row;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  if (threadIdx.x == 0) {
+    const int r = seq_of_token[t], begin = q_start[r], slot = state_slots[r];
+    int token = tokens[t];
+    if (token < 0 || token >= vocab) {
+      atomicOr(status, SPROUT_STATUS_BAD_TOKEN);
+      token = 0;
+    }
+    const bool slot_ok = slot >= 0 && slot < num_slots;
+    if (!slot_ok) atomicOr(status, SPROUT_STATUS_BAD_PAGE);
+    int row = buckets;
+    if (positions[t] > 0) {
+      const long long before = t > begin ? tokens[t - 1] : slot_ok ? last_token[slot] : 0;
+      const long long mixed = (before * mul_prev + token * mul_cur) % buckets;
+      row = (int)(mixed < 0 ? mixed + buckets : mixed);
+    }
+    if (t == begin && slot_ok) last_token[slot] = tokens[q_start[r + 1] - 1];
+    s_token = token;
+    s_row = row;
+  }
+  __syncthreads();
+  const TW* a = table + (size_t)s_token * hidden;
+  const TW* b = pairs + (size_t)s_row * hidden;
+  float* dst = out + (size_t)t * hidden;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = to_float(a[i]) * scale + to_float(b[i]);
+}
+
+SPROUT_API int sprout_embed_pairs(const void* table, const void* pairs, int table_dtype, const int* tokens, const int* positions,
+                                  const int* seq_of_token, const int* q_start, const int* state_slots, int* last_token, int num_slots,
+                                  float* out, int num_tokens, int hidden, int vocab, float scale, long long mul_prev,
+                                  long long mul_cur, int buckets, int* status, cudaStream_t stream) {
+  SPROUT_REQUIRE(num_tokens > 0 && hidden > 0 && vocab > 0 && buckets > 0 && num_slots > 0, "embed_pairs: sizes must be positive");
+  SPROUT_REQUIRE(table && pairs && tokens && positions && seq_of_token && q_start && state_slots && last_token && out && status,
+                 "embed_pairs: null pointer");
+  if (table_dtype == SPROUT_F32)
+    sprout_launch(embed_pairs_kernel<float>, dim3(num_tokens), dim3(256), 0, stream, (const float*)table, (const float*)pairs, tokens,
+                  positions, seq_of_token, q_start, state_slots, last_token, num_slots, out, hidden, vocab, scale, mul_prev, mul_cur,
+                  buckets, status);
+  else if (table_dtype == SPROUT_BF16)
+    sprout_launch(embed_pairs_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(256), 0, stream, (const __nv_bfloat16*)table,
+                  (const __nv_bfloat16*)pairs, tokens, positions, seq_of_token, q_start, state_slots, last_token, num_slots, out,
+                  hidden, vocab, scale, mul_prev, mul_cur, buckets, status);
+  else
+    return sprout_fail("embed_pairs: unknown dtype %d", table_dtype);
+  return sprout_check_launch("embed_pairs");
+}
+
 // ---------------------------------------------------------------- RMSNorm
 // out[r, i] = (x[src(r), i] * rsqrt(mean(x^2) + eps)) * gain[i]; the normalised value is
 // rounded to float32 before the gain multiplies it.  `rows`, when given, selects source rows

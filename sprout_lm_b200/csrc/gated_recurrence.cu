@@ -7,6 +7,8 @@
 //                    per key channel (gated linear attention): a_t[i] = sigmoid(z_t[i] + bias[i])^(1/tau), c_t = 1;
 //                    per head (a selective state space):      dt = softplus(z_t[h] + bias[h]), a_t[i] = exp(-exp(a_log[h]) dt),
 //                                                             c_t = dt;
+//                    a floor (a forget gate that also decides what is written): w_t[i] = (1 - floor[i]) sigmoid(-(z_t[i] + bias[i])),
+//                                                             a_t[i] = 1 - w_t[i]; w_t takes the place of c_t k_t;
 //                    given (a matrix memory with exponential gates): a_t and c_t per head come ready-made from the
 //                                                             caller (`da`, `dc`), whatever the portion's length.
 //                  With `ones_col` the value row gets one more column that is always 1 (column `v_cols` of the state
@@ -19,7 +21,7 @@
 //                  sequence; the last taps - 1 inputs of a request live in its state slot [taps - 1, channels] and are
 //                  read at the start of a portion and replaced at its end.
 //  * gated_group_norm: rows in `groups` equal parts, each divided by its own root mean square, times a weight that
-//                  repeats every `period` elements, times act(gate) before or after the norm.
+//                  repeats every `period` elements, times act(gate) before or after the norm (or without a gate).
 //  * scaled_sum:   x += a y_1 + b y_2.
 #include "common.cuh"
 
@@ -29,7 +31,10 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + lo
 __device__ __forceinline__ float silu_g(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_g(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-enum ScanDecay : int { DECAY_PER_CHANNEL = 0, DECAY_PER_HEAD = 1, DECAY_GIVEN = 2 };
+enum ScanDecay : int { DECAY_PER_CHANNEL = 0, DECAY_PER_HEAD = 1, DECAY_GIVEN = 2, DECAY_FLOOR = 3 };
+
+// What a forget gate with a floor writes: 1 - f for f = floor + (1 - floor) sigmoid(z).
+__device__ __forceinline__ float write_share(float z, float floor) { return (1.0f - floor) * sigmoid_g(-z); }
 
 template <typename T>
 struct ScanParams {
@@ -38,7 +43,7 @@ struct ScanParams {
   const T* v; int v_stride;            // [tokens, heads * vdim]
   const void* z; int z_stride, z_f32;  // per channel: [tokens, heads * dim]; per head: [tokens, heads]; of T, or float when z_f32
   const float* bias;                   // added to z: [heads * dim] or [heads]
-  const float* a_log;                  // per head (per-head decay only)
+  const float* a_log;                  // per head (per-head decay only); with a floor: the floors [heads * dim]
   const float* skip;                   // per head, or null
   float inv_tau, q_scale;
   int mode, heads, groups, dim, vdim;
@@ -51,6 +56,7 @@ struct ScanParams {
   float* sums;                         // [max_chunks, heads, dim, vdim]: a chunk's own sums, then the state before the chunk
   float* prods;                        // [max_chunks, heads, dim]: the product of a chunk's decays
   int chunk, requests;
+  int q_silu;                          // silu on the query rows
   int v_cols, ones_col;                // columns the value rows really have (<= vdim); column v_cols of the state is fed 1
 };
 
@@ -117,7 +123,8 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
     return;
   }
   const int g = h / (p.heads / p.groups);
-  const bool per_head = p.mode != DECAY_PER_CHANNEL;
+  const bool floored = p.mode == DECAY_FLOOR;         // a decay per channel, and no keys
+  const bool per_head = p.mode != DECAY_PER_CHANNEL && !floored;
   float* mine = p.state + (((size_t)slot * p.heads + h) * dim) * p.vdim;
   // the chunk's place in the scratch: the blocks before it belong to the requests before r and to r's earlier chunks
   float* held = PHASE == SCAN_WHOLE ? nullptr : p.sums + (((size_t)(blockIdx.x) * p.heads + h) * dim) * p.vdim;
@@ -161,7 +168,7 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
       if (PHASE != SCAN_WHOLE) rc[u] = 0.f;
       if (tt < n && i < dim) {
         if (PHASE != SCAN_CHUNK_SUMS) rq[u] = to_float(qrow[tt * p.q_stride + i]);
-        rk[u] = to_float(krow[tt * p.k_stride + i]);
+        rk[u] = floored ? 0.f : to_float(krow[tt * p.k_stride + i]);
         if (PHASE == SCAN_WHOLE) {
           const size_t t = tb + tt;
           rz[u] = per_head ? z_at(t * p.z_stride + h) : z_at(t * p.z_stride + (size_t)h * dim + i);
@@ -194,12 +201,14 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
         } else if (per_head) {
           step = softplus_f(rz[u] + p.bias[h]);
           decay = expf(-rate * step);
+        } else if (floored) {
+          decay = write_share(rz[u] + p.bias[(size_t)h * dim + i], p.a_log[(size_t)h * dim + i]);
         } else {
           decay = expf(-softplus_f(-(rz[u] + p.bias[(size_t)h * dim + i])) * p.inv_tau);  // sigmoid(z)^(1/tau) through its logarithm
         }
-        x.x = rq[u] * p.q_scale;
-        x.y = rk[u] * step;
-        x.z = decay;
+        x.x = (p.q_silu ? silu_g(rq[u]) : rq[u]) * p.q_scale;
+        x.y = floored ? decay : rk[u] * step;
+        x.z = floored ? 1.0f - decay : decay;
       }
       tok[e] = x;
     }
@@ -278,7 +287,7 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
 }
 
 // The decays of every token of the step, once: per key channel a = sigmoid(z + bias)^(1 / tau); per head
-// dt = softplus(z + bias), a = exp(-exp(a_log) dt), c = dt.
+// dt = softplus(z + bias), a = exp(-exp(a_log) dt), c = dt; with a floor what is written, 1 - a (`a_log` holds the floors).
 __global__ void scan_decay_kernel(const void* __restrict__ z, int z_stride, int z_f32, int is_bf16, const float* __restrict__ bias,
                                   const float* __restrict__ a_log, float inv_tau, int mode, int heads, int dim, long long count,
                                   float* __restrict__ da, float* __restrict__ dc) {
@@ -294,6 +303,8 @@ __global__ void scan_decay_kernel(const void* __restrict__ z, int z_stride, int 
       const float step = softplus_f(zv + bias[c]);
       da[e] = expf(-expf(a_log[c]) * step);
       dc[e] = step;
+    } else if (mode == DECAY_FLOOR) {
+      da[e] = write_share(zv + bias[c], a_log[c]);
     } else {
       da[e] = expf(-softplus_f(-(zv + bias[c])) * inv_tau);
     }
@@ -417,7 +428,7 @@ gated_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate,
   pdl_wait();
   const int part = width / groups, base = blockIdx.y * part;
   const float* src = o + (size_t)blockIdx.x * width + base;
-  const T* grow = gate + (size_t)blockIdx.x * gate_stride + base;
+  const T* grow = gate ? gate + (size_t)blockIdx.x * gate_stride + base : nullptr;
   float q = 0.f;
   for (int i = threadIdx.x; i < part; i += blockDim.x) {
     float v = src[i];
@@ -430,8 +441,8 @@ gated_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate,
   const float r = 1.0f / sqrtf(block_sum(q, scratch) / (float)part + eps);
   T* dst = out + (size_t)blockIdx.x * width + base;
   for (int i = threadIdx.x; i < part; i += blockDim.x) {
-    const float gv = to_float(grow[i]);
-    const float factor = act ? silu_g(gv) : sigmoid_g(gv);
+    const float gv = grow ? to_float(grow[i]) : 0.f;
+    const float factor = !grow ? 1.0f : act ? silu_g(gv) : sigmoid_g(gv);
     const float v = gate_first ? (src[i] * factor) * r * weight[(base + i) % period] : src[i] * r * weight[(base + i) % period] * factor;
     dst[i] = from_float<T>(v);
   }
@@ -494,8 +505,8 @@ SPROUT_API int sprout_gated_scan(const void* q, int q_stride, const void* k, int
                                  float inv_tau, float q_scale, int mode, int requests, int heads, int groups, int dim, int vdim,
                                  const int* q_start, const int* state_slots, float* state, int num_slots, float* out, int* status,
                                  int tokens, int chunk, int max_chunks, float* da, float* dc, float* sums, float* prods,
-                                 int v_cols, int ones_col, cudaStream_t stream) {
-  SPROUT_REQUIRE(q && k && v && q_start && state_slots && state && out && status, "gated_scan: null pointer");
+                                 int v_cols, int ones_col, int q_silu, cudaStream_t stream) {
+  SPROUT_REQUIRE(q && (k || mode == DECAY_FLOOR) && v && q_start && state_slots && state && out && status, "gated_scan: null pointer");
   SPROUT_REQUIRE(mode == DECAY_GIVEN ? (da && dc) : (z && bias), "gated_scan: the decay's inputs are missing");
   SPROUT_REQUIRE(v_cols > 0 && v_cols <= vdim && (!ones_col || v_cols < vdim), "gated_scan: the value rows' columns do not fit the state's");
   if (mode == DECAY_GIVEN && !sums) {
@@ -515,19 +526,20 @@ SPROUT_API int sprout_gated_scan(const void* q, int q_stride, const void* k, int
   }
   SPROUT_REQUIRE(requests > 0 && heads > 0 && groups > 0 && heads % groups == 0 && dim > 0 && vdim > 0 && num_slots > 0,
                  "gated_scan: bad sizes");
-  SPROUT_REQUIRE(mode == DECAY_PER_CHANNEL || (mode == DECAY_PER_HEAD && a_log) || mode == DECAY_GIVEN, "gated_scan: unknown decay form");
+  SPROUT_REQUIRE(mode == DECAY_PER_CHANNEL || ((mode == DECAY_PER_HEAD || mode == DECAY_FLOOR) && a_log) || mode == DECAY_GIVEN, "gated_scan: unknown decay form");
+  SPROUT_REQUIRE(mode != DECAY_FLOOR || groups == heads, "gated_scan: a forget gate with a floor has query vectors per head");
   SPROUT_REQUIRE(heads <= 65535, "gated_scan: too many heads");
   if (dtype == SPROUT_F32) {
     ScanParams<float> p{(const float*)q, q_stride, (const float*)k, k_stride, (const float*)v, v_stride, z, z_stride, z_f32,
                         bias, a_log, skip, inv_tau, q_scale, mode, heads, groups, dim, vdim, q_start, state_slots, state,
-                        num_slots, out, status, da, dc, sums, prods, chunk, requests, v_cols, ones_col};
+                        num_slots, out, status, da, dc, sums, prods, chunk, requests, q_silu, v_cols, ones_col};
     return launch_scan(p, requests, max_chunks, stream);
   }
   if (dtype == SPROUT_BF16) {
     ScanParams<__nv_bfloat16> p{(const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, k_stride, (const __nv_bfloat16*)v,
                                 v_stride, z, z_stride, z_f32, bias, a_log, skip, inv_tau, q_scale, mode, heads,
                                 groups, dim, vdim, q_start, state_slots, state, num_slots, out, status, da, dc, sums, prods, chunk,
-                                requests, v_cols, ones_col};
+                                requests, q_silu, v_cols, ones_col};
     return launch_scan(p, requests, max_chunks, stream);
   }
   return sprout_fail("gated_scan: unknown dtype %d", dtype);
@@ -557,8 +569,8 @@ SPROUT_API int sprout_causal_conv(const void* in, int in_stride, const float* we
 SPROUT_API int sprout_gated_group_norm(const float* o, const void* gate, int gate_stride, const float* weight, int period, void* out,
                                        int dtype, int rows, int width, int groups, float eps, int gate_first, int act,
                                        cudaStream_t stream) {
-  SPROUT_REQUIRE(o && gate && weight && out && rows > 0 && width > 0 && eps > 0, "gated_group_norm: bad arguments");
-  SPROUT_REQUIRE(groups > 0 && groups <= 65535 && width % groups == 0 && period > 0 && gate_stride >= width,
+  SPROUT_REQUIRE(o && (gate || !gate_first) && weight && out && rows > 0 && width > 0 && eps > 0, "gated_group_norm: bad arguments");
+  SPROUT_REQUIRE(groups > 0 && groups <= 65535 && width % groups == 0 && period > 0 && (!gate || gate_stride >= width),
                  "gated_group_norm: the row must divide into the groups, gate rows must hold the row");
   if (dtype == SPROUT_F32)
     sprout_launch(gated_group_norm_kernel<float>, dim3(rows, groups), dim3(128), 0, stream, o, (const float*)gate, gate_stride, weight,

@@ -10,10 +10,13 @@
 //
 //  * rope_maps_append:          rotates the first `rot` elements of every query and key vector by the
 //                               token's position (half-split pairs) and appends keys and values to the cache; before
-//                               the rotation it can divide every vector by its root mean square and multiply it by a
-//                               weight (one for queries, one for keys).
+//                               the rotation it can divide every vector (or all queries of the token at once, and all
+//                               keys) by its root mean square and multiply it by a weight (one for queries, one for
+//                               keys).  Pairs are (i, i + half) or (2i, 2i + 1).  With tables for the values it also
+//                               turns every value row by its position before it is cached.
 // Options of both attention kernels: a mask (a window, a window that also keeps the first positions, chunks), a cap on
-// the scaled scores (cap * tanh(score / cap)), a sink per head in the softmax denominator, a gate per head.
+// the scaled scores (cap * tanh(score / cap)), a sink per head in the softmax denominator, a gate per head or per element
+// of the output, and for values that were turned by their position a turn of every head's output back by the query's.
 //  * multimap_attention_simple: one block per (token, query head); keys in chunks of 128 aligned to
 //                               absolute position with running maxima and sums: what is done for a query
 //                               does not depend on how the tokens were cut into steps.
@@ -47,7 +50,9 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
                         T* __restrict__ k_cache, T* __restrict__ v_cache, int q_vectors, int kv_heads, int maps, int dim,
                         int rot, int vdim, int page_tokens, int num_pages, int write, float unit_eps, int value_from_key,
                         const float* __restrict__ q_weight, const float* __restrict__ k_weight, float weight_eps,
+                        int weight_whole, int interleaved, const float* __restrict__ v_cos, const float* __restrict__ v_sin,
                         int* status) {
+  __shared__ float norm_scratch[33];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -68,15 +73,31 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
   }
   const int kw = maps * dim;
   const int vectors = q_vectors + (write ? kv_heads * maps : 0);
+  // a norm over the whole projection: one factor for all query vectors of the token, one for all its key vectors
+  float whole_q = 1.0f, whole_k = 1.0f;
+  if (weight_whole) {
+    auto root = [&](const T* src, int count) {
+      float sq = 0.f;
+      for (int i = threadIdx.x; i < count; i += blockDim.x) {
+        const float x = to_float(src[i]);
+        sq = fmaf(x, x, sq);
+      }
+      return 1.0f / sqrtf(block_sum(sq, norm_scratch) / (float)count + weight_eps);
+    };
+    if (q_weight != nullptr) whole_q = root(row, q_vectors * dim);
+    if (k_weight != nullptr && write) whole_k = root(row + (size_t)q_vectors * dim, kv_heads * kw);
+    __syncthreads();                                              // every element was read before any is rewritten
+  }
   for (int vec = warp; vec < vectors; vec += warps) {
     const bool is_key = vec >= q_vectors;
     if (is_key && page < 0) continue;
     const float* weight = is_key ? k_weight : q_weight;           // the norm before the rotation, when the vector has one
+    if (weight_whole && weight != nullptr) weight += (size_t)(is_key ? vec - q_vectors : vec) * dim;
     if (!is_key && !turn && unit_eps <= 0.f && weight == nullptr) continue;   // nothing to do to this query vector
     T* src = row + (size_t)vec * dim;                             // the key vectors follow the query vectors
     float vals[ROPE_MAX_PER_LANE], raw[ROPE_MAX_PER_LANE];
-    float before = 1.0f;
-    if (weight != nullptr) {
+    float before = is_key ? whole_k : whole_q;
+    if (weight != nullptr && !weight_whole) {
       float sq = 0.f;
 #pragma unroll
       for (int j = 0; j < ROPE_MAX_PER_LANE; j++)
@@ -96,10 +117,11 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
         raw[j] = x;
         if (weight != nullptr) x = x * before * weight[d];
         if (turn && d < rot) {
-          const int i = d < half ? d : d - half, partner = d < half ? d + half : d - half;
+          const bool leads = interleaved ? (d & 1) == 0 : d < half;     // the first element of its pair
+          const int i = interleaved ? d >> 1 : leads ? d : d - half, partner = interleaved ? d ^ 1 : leads ? d + half : d - half;
           float other = to_float(src[partner]);
           if (weight != nullptr) other = other * before * weight[partner];
-          x = d < half ? x * cs[i] - other * sn[i] : x * cs[i] + other * sn[i];
+          x = leads ? x * cs[i] - other * sn[i] : x * cs[i] + other * sn[i];
         }
         vals[j] = x;
         squares = fmaf(x, x, squares);
@@ -127,6 +149,24 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
   }
   if (!write || page < 0 || value_from_key) return;
   const T* vrow = row + (size_t)q_vectors * dim + (size_t)kv_heads * kw;
+  if (v_cos != nullptr) {
+    // values turned by their position over all of their elements, in the same layout of pairs
+    if (pos >= max_positions) {
+      if (threadIdx.x == 0) atomicOr(status, SPROUT_STATUS_BAD_POSITION);
+      return;
+    }
+    const int vhalf = vdim / 2;
+    for (int i = threadIdx.x; i < kv_heads * vhalf; i += blockDim.x) {
+      const int g = i / vhalf, m = i % vhalf;
+      const int e0 = interleaved ? 2 * m : m, e1 = interleaved ? 2 * m + 1 : m + vhalf;
+      const float c = v_cos[(size_t)pos * vhalf + m], s = v_sin[(size_t)pos * vhalf + m];
+      const float a = to_float(vrow[g * vdim + e0]), b = to_float(vrow[g * vdim + e1]);
+      T* dst = v_cache + (((size_t)page * kv_heads + g) * page_tokens + pos % page_tokens) * vdim;
+      dst[e0] = from_float<T>(a * c - b * s);
+      dst[e1] = from_float<T>(b * c + a * s);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < kv_heads * vdim; i += blockDim.x) {
     const int g = i / vdim, e = i % vdim;
     v_cache[(((size_t)page * kv_heads + g) * page_tokens + pos % page_tokens) * vdim + e] = vrow[i];
@@ -148,6 +188,12 @@ __device__ __forceinline__ int first_visible(int kind, int size, int pos) {
   return 0;
 }
 
+// Turns a head's output back by the query's position (values that were turned by theirs): tables float32
+// [positions, vdim / 2]; null: no turn.  Pair m is (m, m + vdim / 2), or (2m, 2m + 1) when `interleaved`.
+struct OutputTurn {
+  const float* cos; const float* sin; int positions, interleaved;
+};
+
 template <typename T, int MAPS>
 __global__ void __launch_bounds__(CHUNK)
 multimap_attention_simple_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ k_cache,
@@ -156,7 +202,8 @@ multimap_attention_simple_kernel(const T* __restrict__ q, int q_stride, const T*
                                  T* __restrict__ out, int out_stride, int heads, int kv_heads, int dim, int vdim,
                                  int page_tokens, int num_pages, float scale, float lambda, float norm_eps,
                                  float out_scale, int mask_kind, int mask_size, int mask_keep, float softcap,
-                                 const float* __restrict__ sink, const T* __restrict__ gate, int gate_stride, int* status) {
+                                 const float* __restrict__ sink, const T* __restrict__ gate, int gate_stride, int gate_elements,
+                                 const OutputTurn turn, int* status) {
   extern __shared__ float smem[];
   float* qs = smem;                                   // MAPS * dim
   float* probs = qs + MAPS * dim;                     // MAPS * CHUNK
@@ -262,11 +309,34 @@ multimap_attention_simple_kernel(const T* __restrict__ q, int q_stride, const T*
   }
   float factor = out_scale;
   if (norm_eps > 0.f) factor *= 1.0f / sqrtf(block_sum(squares, scratch) / (float)vdim + norm_eps);
-  if (gate != nullptr) factor *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + h])));
+  if (turn.cos != nullptr) {
+    float* whole = (float*)(row_index + CHUNK);       // vdim
+#pragma unroll
+    for (int part = 0; part < PARTS; part++)
+      if (tid + part * CHUNK < vdim) whole[tid + part * CHUNK] = o[part];
+    __syncthreads();
+    const int half = vdim / 2;
+    const size_t at = (size_t)min(max(pos, 0), turn.positions - 1) * half;
+#pragma unroll
+    for (int part = 0; part < PARTS; part++) {
+      const int e = tid + part * CHUNK;
+      if (e >= vdim) continue;
+      const bool leads = turn.interleaved ? (e & 1) == 0 : e < half;
+      const int m = turn.interleaved ? e >> 1 : leads ? e : e - half;
+      const float other = whole[turn.interleaved ? e ^ 1 : leads ? e + half : e - half], c = turn.cos[at + m], s = turn.sin[at + m];
+      o[part] = leads ? o[part] * c + other * s : o[part] * c - other * s;
+    }
+  }
+  if (gate != nullptr && !gate_elements) factor *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + h])));
+  const T* gates = gate != nullptr && gate_elements ? gate + (size_t)t * gate_stride + (size_t)h * vdim : nullptr;
   T* dst = out + (size_t)t * out_stride + (size_t)h * vdim;
 #pragma unroll
   for (int part = 0; part < PARTS; part++)
-    if (tid + part * CHUNK < vdim) dst[tid + part * CHUNK] = from_float<T>(o[part] * factor);
+    if (tid + part * CHUNK < vdim) {
+      float v = o[part] * factor;
+      if (gates) v *= 1.0f / (1.0f + expf(-to_float(gates[tid + part * CHUNK])));
+      dst[tid + part * CHUNK] = from_float<T>(v);
+    }
 }
 
 
@@ -290,7 +360,14 @@ struct MultiMapParams {
   int mask_kind, mask_size; const float* sink; const __nv_bfloat16* gate; int gate_stride;
   // a window's kept first positions, and the cap on the scaled scores (0: none)
   int mask_keep; float softcap;
+  // the gate row holds a number per element of the output instead of one per head; the turn back of the output
+  int gate_elements; OutputTurn turn;
 };
+
+// A gate per element: sigmoid of the gate row's number for column `col` of the head's output.
+__device__ __forceinline__ float element_gate(const MultiMapParams& p, int token, int head, int vdim, int col) {
+  return 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(size_t)token * p.gate_stride + (size_t)head * vdim + col])));
+}
 
 // What the running maxima are multiplied by on their way into the exponentials: capped scores are already scaled.
 __device__ __forceinline__ float score_scale(const MultiMapParams& p) { return p.softcap > 0.f ? 1.0f : p.scale; }
@@ -631,7 +708,40 @@ multimap_attention_mma_kernel(const MultiMapParams p) {
     f0 *= 1.0f / sqrtf(sq0 / (float)VDIM + p.norm_eps);
     f1 *= 1.0f / sqrtf(sq1 / (float)VDIM + p.norm_eps);
   }
-  if (p.gate != nullptr) {
+  if (p.turn.cos != nullptr) {
+    // back by the query's position, on the accumulators: both elements of a pair are this thread's
+    const size_t at0 = (size_t)min(max(limit0, 0), p.turn.positions - 1) * (VDIM / 2), at1 = (size_t)min(max(limit1, 0), p.turn.positions - 1) * (VDIM / 2);
+    if (p.turn.interleaved) {
+#pragma unroll
+      for (int i = 0; i < VDIM / 8; i++) {
+        const int m = i * 4 + qc;
+        const float c0 = p.turn.cos[at0 + m], s0 = p.turn.sin[at0 + m], c1 = p.turn.cos[at1 + m], s1 = p.turn.sin[at1 + m];
+        const float a0 = o[0][i][0], b0 = o[0][i][1], a1 = o[0][i][2], b1 = o[0][i][3];
+        o[0][i][0] = a0 * c0 + b0 * s0; o[0][i][1] = b0 * c0 - a0 * s0;
+        o[0][i][2] = a1 * c1 + b1 * s1; o[0][i][3] = b1 * c1 - a1 * s1;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < VDIM / 16; i++)
+#pragma unroll
+        for (int c = 0; c < 2; c++) {
+          const int m = i * 8 + qc * 2 + c;
+          const float c0 = p.turn.cos[at0 + m], s0 = p.turn.sin[at0 + m], c1 = p.turn.cos[at1 + m], s1 = p.turn.sin[at1 + m];
+          const float a0 = o[0][i][c], b0 = o[0][i + VDIM / 16][c], a1 = o[0][i][2 + c], b1 = o[0][i + VDIM / 16][2 + c];
+          o[0][i][c] = a0 * c0 + b0 * s0; o[0][i + VDIM / 16][c] = b0 * c0 - a0 * s0;
+          o[0][i][2 + c] = a1 * c1 + b1 * s1; o[0][i + VDIM / 16][2 + c] = b1 * c1 - a1 * s1;
+        }
+    }
+  }
+  if (p.gate != nullptr && p.gate_elements) {
+#pragma unroll
+    for (int i = 0; i < VDIM / 8; i++)
+#pragma unroll
+      for (int c = 0; c < 2; c++) {
+        if (s_token[my_row0] >= 0) o[0][i][c] *= element_gate(p, s_token[my_row0], s_head[my_row0], VDIM, i * 8 + qc * 2 + c);
+        if (s_token[my_row1] >= 0) o[0][i][2 + c] *= element_gate(p, s_token[my_row1], s_head[my_row1], VDIM, i * 8 + qc * 2 + c);
+      }
+  } else if (p.gate != nullptr) {
     if (s_token[my_row0] >= 0) f0 *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(size_t)s_token[my_row0] * p.gate_stride + s_head[my_row0]])));
     if (s_token[my_row1] >= 0) f1 *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(size_t)s_token[my_row1] * p.gate_stride + s_head[my_row1]])));
   }
@@ -652,6 +762,7 @@ template <int MAPS>
 __global__ void __launch_bounds__(128)
 multimap_merge_kernel(const MultiMapParams p, int vdim) {
   __shared__ float scratch[33];
+  __shared__ float whole[256];
   pdl_launch_dependents();
   pdl_wait();
   const int r = blockIdx.x, g = blockIdx.y, row = blockIdx.z, group = p.heads / p.kv_heads;
@@ -690,7 +801,30 @@ multimap_merge_kernel(const MultiMapParams p, int vdim) {
     if (threadIdx.x + part * 128 < vdim) squares = fmaf(v[part], v[part], squares);
   float factor = p.out_scale;
   if (p.norm_eps > 0.f) factor *= 1.0f / sqrtf(block_sum(squares, scratch) / (float)vdim + p.norm_eps);
-  if (p.gate != nullptr) factor *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(size_t)token * p.gate_stride + head])));
+  if (p.turn.cos != nullptr) {
+#pragma unroll
+    for (int part = 0; part < 2; part++)
+      if (threadIdx.x + part * 128 < vdim) whole[threadIdx.x + part * 128] = v[part];
+    __syncthreads();
+    const int half = vdim / 2;
+    const size_t at = (size_t)min(max(p.positions[token], 0), p.turn.positions - 1) * half;
+#pragma unroll
+    for (int part = 0; part < 2; part++) {
+      const int e = threadIdx.x + part * 128;
+      if (e >= vdim) continue;
+      const bool leads = p.turn.interleaved ? (e & 1) == 0 : e < half;
+      const int m = p.turn.interleaved ? e >> 1 : leads ? e : e - half;
+      const float other = whole[p.turn.interleaved ? e ^ 1 : leads ? e + half : e - half], c = p.turn.cos[at + m], s = p.turn.sin[at + m];
+      v[part] = leads ? v[part] * c + other * s : v[part] * c - other * s;
+    }
+  }
+  if (p.gate != nullptr && p.gate_elements) {
+#pragma unroll
+    for (int part = 0; part < 2; part++)
+      if (threadIdx.x + part * 128 < vdim) v[part] *= element_gate(p, token, head, vdim, threadIdx.x + part * 128);
+  } else if (p.gate != nullptr) {
+    factor *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(size_t)token * p.gate_stride + head])));
+  }
   __nv_bfloat16* dst = p.out + (size_t)token * p.out_stride + (size_t)head * vdim;
 #pragma unroll
   for (int part = 0; part < 2; part++)
@@ -720,7 +854,8 @@ int launch_multimap(const MultiMapParams& p, int grid_x, cudaStream_t stream) {
 
 bool mma_sizes(int maps, int dim, int vdim) {
   return (maps == 1 || maps == 2) && ((dim == 32 && vdim == 64) || (dim == 64 && vdim == 64) || (dim == 64 && vdim == 128) ||
-                                      (dim == 128 && vdim == 128) || (dim == 16 && vdim == 32) || (dim == 32 && vdim == 32));
+                                      (dim == 128 && vdim == 128) || (dim == 16 && vdim == 32) || (dim == 32 && vdim == 32) ||
+                                      (maps == 1 && ((dim == 96 && vdim == 96) || (dim == 48 && vdim == 48) || (dim == 80 && vdim == 80))));
 }
 
 }  // namespace
@@ -740,8 +875,9 @@ SPROUT_API int sprout_multimap_attention_mma(const void* q, int q_stride, const 
                                              int max_q_len, int heads, int kv_heads, int maps, int dim, int vdim, int page_tokens,
                                              int num_pages, float scale, float lambda, float norm_eps, float out_scale,
                                              int ksplit, float* partial, int mask_kind, int mask_size, const float* sink,
-                                             const void* gate, int gate_stride, int mask_keep, float softcap, int* status,
-                                             cudaStream_t stream) {
+                                             const void* gate, int gate_stride, int mask_keep, float softcap, int gate_elements,
+                                             const float* turn_cos, const float* turn_sin, int turn_positions, int turn_interleaved,
+                                             int* status, cudaStream_t stream) {
   SPROUT_REQUIRE(q && k_cache && v_cache && block_table && q_start && positions && out && status, "multimap_attention_mma: null pointer");
   SPROUT_REQUIRE(requests > 0 && tiles > 0 && max_q_len > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && page_tokens > 0 &&
                  num_pages > 0, "multimap_attention_mma: bad sizes");
@@ -752,12 +888,14 @@ SPROUT_API int sprout_multimap_attention_mma(const void* q, int q_stride, const 
   MultiMapParams p{(const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, block_table,
                    table_stride, q_start, positions, (__nv_bfloat16*)out, out_stride, requests, heads, kv_heads, page_tokens,
                    num_pages, scale, lambda, norm_eps, out_scale, status, ksplit, partial, mask_kind, mask_size, sink,
-                   (const __nv_bfloat16*)gate, gate_stride, mask_keep, softcap};
+                   (const __nv_bfloat16*)gate, gate_stride, mask_keep, softcap, gate_elements,
+                   {turn_cos, turn_sin, turn_positions, turn_interleaved}};
+  SPROUT_REQUIRE(!turn_cos || (turn_sin && turn_positions > 0), "multimap_attention_mma: the turn's tables are missing");
   SPROUT_REQUIRE(mask_kind == MASK_CAUSAL || ((mask_kind == MASK_WINDOW || mask_kind == MASK_CHUNK) && mask_size > 0),
                  "multimap_attention_mma: a window or a chunk needs a positive size");
   SPROUT_REQUIRE(mask_keep >= 0 && (mask_keep == 0 || mask_kind == MASK_WINDOW) && softcap >= 0.f,
                  "multimap_attention_mma: only a window keeps first positions; the cap is not negative");
-  SPROUT_REQUIRE(!gate || gate_stride >= heads, "multimap_attention_mma: gate rows hold a number per head");
+  SPROUT_REQUIRE(!gate || gate_stride >= (gate_elements ? heads * vdim : heads), "multimap_attention_mma: gate rows hold a number per head or element");
   SPROUT_REQUIRE(ksplit >= 1 && ksplit <= 64 && (ksplit == 1 || (partial && max_q_len * (heads / kv_heads) <= 16)),
                  "multimap_attention_mma: keys are divided among CTAs in single-token steps only, with scratch for the shares");
   const bool split = max_q_len * (heads / kv_heads) <= 16;
@@ -768,6 +906,11 @@ SPROUT_API int sprout_multimap_attention_mma(const void* q, int q_stride, const 
   }
   PICK(32, 64) PICK(64, 64) PICK(64, 128) PICK(128, 128) PICK(16, 32) PICK(32, 32)
 #undef PICK
+#define PICK(D, V)                                                                                              \
+  if (dim == D && vdim == V && maps == 1)                                                                       \
+    return split ? launch_multimap<D, V, 1, true>(p, tiles, stream) : launch_multimap<D, V, 1, false>(p, tiles, stream);
+  PICK(96, 96) PICK(48, 48) PICK(80, 80)
+#undef PICK
   return sprout_fail("multimap_attention_mma: no kernel for these sizes");
 }
 
@@ -776,7 +919,8 @@ SPROUT_API int sprout_rope_maps_append(void* rows, int row_stride, int dtype, co
                                        const float* sin_table, int max_positions, void* k_cache, void* v_cache, int tokens,
                                        int q_vectors, int kv_heads, int maps, int dim, int rot, int vdim, int page_tokens,
                                        int num_pages, int write, float unit_eps, int value_from_key, const float* q_weight,
-                                       const float* k_weight, float weight_eps, int* status, cudaStream_t stream) {
+                                       const float* k_weight, float weight_eps, int weight_whole, int interleaved,
+                                       const float* v_cos, const float* v_sin, int* status, cudaStream_t stream) {
   SPROUT_REQUIRE(rows && positions && status && tokens > 0 && q_vectors > 0 && dim > 0 && maps > 0, "rope_maps_append: bad arguments");
   SPROUT_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dim, "rope_maps_append: the rotated width must be even and at most dim");
   SPROUT_REQUIRE(rot == 0 || (cos_table && sin_table && max_positions > 0), "rope_maps_append: tables are missing");
@@ -785,18 +929,19 @@ SPROUT_API int sprout_rope_maps_append(void* rows, int row_stride, int dtype, co
   SPROUT_REQUIRE(dim <= 32 * ROPE_MAX_PER_LANE, "rope_maps_append: vectors of up to %d elements (got %d)", 32 * ROPE_MAX_PER_LANE, dim);
   SPROUT_REQUIRE(!value_from_key || vdim == maps * dim, "rope_maps_append: values that are the keys have the keys' width");
   SPROUT_REQUIRE((!q_weight && !k_weight) || weight_eps > 0.f, "rope_maps_append: a norm before the rotation needs a positive eps");
+  SPROUT_REQUIRE(!v_cos || (v_sin && max_positions > 0 && vdim % 2 == 0 && !value_from_key), "rope_maps_append: values turn in pairs, with tables of their own");
   const int need = q_vectors * dim + (write ? kv_heads * (maps * dim + (value_from_key ? 0 : vdim)) : 0);
   SPROUT_REQUIRE(row_stride >= need, "rope_maps_append: rows of %d elements, %d needed", row_stride, need);
   if (dtype == SPROUT_F32)
     sprout_launch(rope_maps_append_kernel<float>, dim3(tokens), dim3(128), 0, stream, (float*)rows, row_stride, positions,
                   seq_of_token, block_table, table_stride, cos_table, sin_table, max_positions, (float*)k_cache,
                   (float*)v_cache, q_vectors, kv_heads, maps, dim, rot, vdim, page_tokens, num_pages, write, unit_eps,
-                  value_from_key, q_weight, k_weight, weight_eps, status);
+                  value_from_key, q_weight, k_weight, weight_eps, weight_whole, interleaved, v_cos, v_sin, status);
   else if (dtype == SPROUT_BF16)
     sprout_launch(rope_maps_append_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, stream, (__nv_bfloat16*)rows, row_stride,
                   positions, seq_of_token, block_table, table_stride, cos_table, sin_table, max_positions,
                   (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, q_vectors, kv_heads, maps, dim, rot, vdim, page_tokens,
-                  num_pages, write, unit_eps, value_from_key, q_weight, k_weight, weight_eps, status);
+                  num_pages, write, unit_eps, value_from_key, q_weight, k_weight, weight_eps, weight_whole, interleaved, v_cos, v_sin, status);
   else
     return sprout_fail("rope_maps_append: unknown dtype %d", dtype);
   return sprout_check_launch("rope_maps_append");
@@ -808,8 +953,9 @@ SPROUT_API int sprout_multimap_attention_simple(const void* q, int q_stride, con
                                                 int heads, int kv_heads, int maps, int dim, int vdim, int page_tokens,
                                                 int num_pages, float scale, float lambda, float norm_eps, float out_scale,
                                                 int mask_kind, int mask_size, const float* sink, const void* gate,
-                                                int gate_stride, int mask_keep, float softcap, int* status,
-                                                cudaStream_t stream) {
+                                                int gate_stride, int mask_keep, float softcap, int gate_elements,
+                                                const float* turn_cos, const float* turn_sin, int turn_positions,
+                                                int turn_interleaved, int* status, cudaStream_t stream) {
   SPROUT_REQUIRE(q && k_cache && v_cache && block_table && seq_of_token && positions && out && status, "multimap_attention: null pointer");
   SPROUT_REQUIRE(tokens > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && page_tokens > 0 && num_pages > 0,
                  "multimap_attention: bad sizes");
@@ -818,17 +964,19 @@ SPROUT_API int sprout_multimap_attention_simple(const void* q, int q_stride, con
   SPROUT_REQUIRE(heads <= 65535, "multimap_attention: too many heads");
   SPROUT_REQUIRE(mask_kind == MASK_CAUSAL || ((mask_kind == MASK_WINDOW || mask_kind == MASK_CHUNK) && mask_size > 0),
                  "multimap_attention: a window or a chunk needs a positive size");
-  SPROUT_REQUIRE(!gate || gate_stride >= heads, "multimap_attention: gate rows hold a number per head");
+  SPROUT_REQUIRE(!gate || gate_stride >= (gate_elements ? heads * vdim : heads), "multimap_attention: gate rows hold a number per head or element");
+  SPROUT_REQUIRE(!turn_cos || (turn_sin && turn_positions > 0 && vdim % 2 == 0), "multimap_attention: the turn's tables are missing");
+  const OutputTurn turn{turn_cos, turn_sin, turn_positions, turn_interleaved};
   SPROUT_REQUIRE(mask_keep >= 0 && (mask_keep == 0 || mask_kind == MASK_WINDOW) && softcap >= 0.f,
                  "multimap_attention: only a window keeps first positions; the cap is not negative");
-  const size_t smem = (size_t)(maps * dim + maps * CHUNK + 36) * sizeof(float) + CHUNK * sizeof(long long);
+  const size_t smem = (size_t)(maps * dim + maps * CHUNK + 36 + (turn_cos ? vdim : 0)) * sizeof(float) + CHUNK * sizeof(long long);
   SPROUT_REQUIRE(smem <= 48 * 1024, "multimap_attention: key vectors too long (%d)", dim);
   dim3 grid(tokens, heads);
 #define LAUNCH(T, M)                                                                                                      \
   sprout_launch(multimap_attention_simple_kernel<T, M>, grid, dim3(CHUNK), smem, stream, (const T*)q, q_stride,           \
                 (const T*)k_cache, (const T*)v_cache, block_table, table_stride, seq_of_token, positions, (T*)out,        \
                 out_stride, heads, kv_heads, dim, vdim, page_tokens, num_pages, scale, lambda, norm_eps, out_scale,    \
-                mask_kind, mask_size, mask_keep, softcap, sink, (const T*)gate, gate_stride, status)
+                mask_kind, mask_size, mask_keep, softcap, sink, (const T*)gate, gate_stride, gate_elements, turn, status)
   if (dtype == SPROUT_F32) {
     if (maps == 1) LAUNCH(float, 1); else LAUNCH(float, 2);
   } else if (dtype == SPROUT_BF16) {

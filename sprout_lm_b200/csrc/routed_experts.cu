@@ -6,15 +6,17 @@
 //                  `experts` on are identity experts (their output is the token's h).  Counts the rows
 //                  of each real expert.  Options: the outputs form `group_count` equal groups of neighbours, a group's
 //                  score is its largest s, and only outputs of the `group_keep` best groups can be taken; weights that
-//                  are the scores themselves (not renormalised); `extra` further rows of the router matrix whose
+//                  are the scores themselves (not renormalised); scores that are sigmoids of the single products instead of a
+//                  softmax over them; `extra` further rows of the router matrix whose
 //                  products are handed out as they are (a gate beside the router, in the same 32-bit product).
 //  * moe_arrange:  offsets of the experts' row ranges, every taken (token, place) of a real expert put
 //                  into its expert's range (`sorted`), and where it went (`place_of`).
 //  * moe_up / moe_down (plain): the experts' two products on CUDA cores over the arranged rows, every
 //                  output element summed in ascending k by one warp: act = f(W_gate a, W_up a),
 //                  rows = W_down act, f(g, u) = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit),
-//                  u' = clamp(u, -limit, limit); or, for experts without a gate, act = gelu(W_up a) (the exact, erf form)
-//                  with a matrix of ff rows per expert.
+//                  u' = clamp(u, -limit, limit); or f(g, u) = silu(g) u; or, for experts without a gate, act = gelu(W_up a)
+//                  (the exact, erf form) with a matrix of ff rows per expert.  A row's routing weight may multiply the
+//                  expert's input: the products are linear, so it multiplies both of them before the activation.
 //  * moe_up / moe_down (mma):   the same two products on tensor cores (bfloat16, `mma.sync.m16n8k16`, float32
 //                  accumulation): a CTA makes 128 arranged rows of one expert x 128 columns, K in steps of 64
 //                  through a three-stage cp.async ring; the tile list follows the experts' row counts on the
@@ -22,7 +24,8 @@
 //                  them, so the activation is applied to the accumulators.
 //  * moe_few:      the same two products for steps of at most 8 tokens (bfloat16): a CTA per (expert, 32 output columns)
 //                  keeps the expert's few rows in shared memory and streams every weight row once for all of them.
-//  * moe_combine:  y[t] += sum over the token's places of weight * (identity ? h[t] : its row).
+//  * moe_combine:  y[t] += sum over the token's places of weight * (identity ? h[t] : its row), or one factor times the
+//                  sum of the rows when the weights went into the experts' inputs.
 #include "attention_bf16.cuh"
 
 using namespace sprout_attn;
@@ -43,7 +46,7 @@ __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const T* __restrict__ h, int h_stride, const float* __restrict__ router, const float* __restrict__ correction,
                  int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ counts, int tokens, int width,
                  int softmax_outputs, int experts, int top, float scale, int extra, float* __restrict__ extra_out,
-                 int group_count, int group_keep, int renormalize) {
+                 int group_count, int group_keep, int renormalize, int sigmoid_scores) {
   extern __shared__ float smem[];
   int outputs = softmax_outputs + extra;              // rows of the router matrix
   float* zs = smem;                                   // ROUTE_TOKENS x outputs: scores
@@ -96,17 +99,19 @@ moe_route_kernel(const T* __restrict__ h, int h_stride, const float* __restrict_
   float* choice = choices + warp * outputs;
   for (int e = lane; e < extra; e += 32) extra_out[(size_t)t * extra + e] = z[softmax_outputs + e];
   outputs = softmax_outputs;                          // from here on: what the softmax is over
-  float top_z = -INFINITY;
-  for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, z[e]);
-  top_z = warp_max(top_z);
-  float sum = 0.f;
-  for (int e = lane; e < outputs; e += 32) sum += expf(z[e] - top_z);
-  sum = warp_sum(sum);
+  float top_z = -INFINITY, sum = 0.f;
+  if (!sigmoid_scores) {
+    for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, z[e]);
+    top_z = warp_max(top_z);
+    for (int e = lane; e < outputs; e += 32) sum += expf(z[e] - top_z);
+    sum = warp_sum(sum);
+  }
   __syncwarp();
   for (int e = lane; e < outputs; e += 32) {
-    const float s = expf(z[e] - top_z) / sum;
+    const float zv = z[e], s = sigmoid_scores ? 1.0f / (1.0f + expf(-zv)) : expf(zv - top_z) / sum;
     z[e] = s;
-    choice[e] = s + (correction ? correction[e] : 0.f);
+    // single sigmoids order as their products do, also where 32 bits round them to the same number
+    choice[e] = sigmoid_scores && !correction && group_keep == group_count ? zv : s + (correction ? correction[e] : 0.f);
   }
   __syncwarp();
   if (group_count > 1 && group_keep < group_count) {
@@ -219,9 +224,12 @@ __device__ __forceinline__ int expert_of(const int* offsets, int experts, int ro
   return lo;
 }
 
-// `limit` <= 0 names an expert without a gate: the exact gelu of its one product.
-__device__ __forceinline__ float glu(float g, float u, float limit, float alpha) {
-  if (limit <= 0.f) return 0.5f * g * (1.0f + erff(g * 0.7071067811865476f));
+// What an expert does with its first products: the clamped gated unit, the exact gelu of one product (an expert without a
+// gate), silu(g) u.
+enum ExpertUnit : int { UNIT_CLAMPED = 0, UNIT_PLAIN = 1, UNIT_SILU = 2 };
+__device__ __forceinline__ float glu(int unit, float g, float u, float limit, float alpha) {
+  if (unit == UNIT_PLAIN) return 0.5f * g * (1.0f + erff(g * 0.7071067811865476f));
+  if (unit == UNIT_SILU) return g / (1.0f + expf(-g)) * u;
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * (1.0f / (1.0f + expf(-alpha * g))) * (u + 1.0f);
@@ -233,7 +241,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 moe_up_plain_kernel(const T* __restrict__ h, int h_stride, const int* __restrict__ sorted, const int* __restrict__ offsets,
                     const T* __restrict__ w_gate_up, T* __restrict__ act, int experts, int top, int width, int ff,
-                    float limit, float alpha) {
+                    int unit, const float* __restrict__ row_weights, float limit, float alpha) {
   extern __shared__ float a[];          // width
   pdl_launch_dependents();
   pdl_wait();
@@ -244,7 +252,8 @@ moe_up_plain_kernel(const T* __restrict__ h, int h_stride, const int* __restrict
   for (int k = threadIdx.x; k < width; k += blockDim.x) a[k] = to_float(src[k]);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const bool gated = limit > 0.f;                      // else the matrix has ff rows per expert and no up rows
+  const bool gated = unit != UNIT_PLAIN;               // else the matrix has ff rows per expert and no up rows
+  const float weight = row_weights ? row_weights[sorted[row]] : 1.0f;
   const T* w = w_gate_up + (size_t)e * (gated ? 2 : 1) * ff * width;
   for (int j = blockIdx.y * 8 + warp; j < ff; j += gridDim.y * 8) {
     const T* wg = w + (size_t)j * width;
@@ -257,7 +266,7 @@ moe_up_plain_kernel(const T* __restrict__ h, int h_stride, const int* __restrict
     g = warp_sum(g);
     u = warp_sum(u);
     // the products' results are rounded to the activations' type before the activation, as separate products would leave them
-    if (lane == 0) act[(size_t)row * ff + j] = from_float<T>(glu(to_float(from_float<T>(g)), to_float(from_float<T>(u)), limit, alpha));
+    if (lane == 0) act[(size_t)row * ff + j] = from_float<T>(glu(unit, to_float(from_float<T>(g * weight)), to_float(from_float<T>(u * weight)), limit, alpha));
   }
 }
 
@@ -314,7 +323,7 @@ template <int KIND>
 __global__ void __launch_bounds__(GTHREADS)
 moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int* __restrict__ order,
                     const int* __restrict__ offsets, const __nv_bfloat16* __restrict__ w, void* __restrict__ out,
-                    int experts, int top, int N, int K, float limit, float alpha) {
+                    int experts, int top, int N, int K, int unit, const float* __restrict__ row_weights, float limit, float alpha) {
   extern __shared__ __align__(16) unsigned char gemm_smem[];
   typedef __nv_bfloat16 (*Tile)[GSTRIDE];
   __shared__ const __nv_bfloat16* a_rows[GM];
@@ -402,6 +411,7 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int
     for (int half = 0; half < 2; half++) {
       const int row = row0 + wm * 32 + mi * 16 + gr + half * 8;
       if (row >= row_end) continue;
+      const float weight = GATHER && row_weights ? row_weights[order[row]] : 1.0f;
       if (UP) {
         __nv_bfloat16* dst = (__nv_bfloat16*)out + (size_t)row * ff;
 #pragma unroll
@@ -412,9 +422,9 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int
 #pragma unroll
           for (int c = 0; c < 2; c++) {
             // rounded to bfloat16 before the activation, as separate products would leave them
-            const float g = __bfloat162float(__float2bfloat16_rn(acc[mi][ni][half * 2 + c]));
-            const float u = __bfloat162float(__float2bfloat16_rn(acc[mi][ni + 4][half * 2 + c]));
-            v[c] = glu(g, u, limit, alpha);
+            const float g = __bfloat162float(__float2bfloat16_rn(acc[mi][ni][half * 2 + c] * weight));
+            const float u = __bfloat162float(__float2bfloat16_rn(acc[mi][ni + 4][half * 2 + c] * weight));
+            v[c] = glu(unit, g, u, limit, alpha);
           }
           *(__nv_bfloat162*)(dst + j) = __floats2bfloat162_rn(v[0], v[1]);
         }
@@ -425,9 +435,9 @@ moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int
           const int n = n0 + wn * 64 + ni * 8 + qc * 2;
           if (n >= N) continue;
           // rounded to bfloat16 before the activation, as a separate product would leave it
-          const float g0 = __bfloat162float(__float2bfloat16_rn(acc[mi][ni][half * 2]));
-          const float g1 = __bfloat162float(__float2bfloat16_rn(acc[mi][ni][half * 2 + 1]));
-          *(__nv_bfloat162*)(dst + n) = __floats2bfloat162_rn(glu(g0, 0.f, 0.f, 0.f), glu(g1, 0.f, 0.f, 0.f));
+          const float g0 = __bfloat162float(__float2bfloat16_rn(acc[mi][ni][half * 2] * weight));
+          const float g1 = __bfloat162float(__float2bfloat16_rn(acc[mi][ni][half * 2 + 1] * weight));
+          *(__nv_bfloat162*)(dst + n) = __floats2bfloat162_rn(glu(UNIT_PLAIN, g0, 0.f, 0.f, 0.f), glu(UNIT_PLAIN, g1, 0.f, 0.f, 0.f));
         }
       } else {
         float* dst = (float*)out + (size_t)row * N;
@@ -449,7 +459,8 @@ constexpr int FEW = 8, FEW_COLS = 32;
 template <bool UP>
 __global__ void __launch_bounds__(256)
 moe_few_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int* __restrict__ order, const int* __restrict__ offsets,
-               const __nv_bfloat16* __restrict__ w, void* __restrict__ out, int top, int N, int K, float limit, float alpha) {
+               const __nv_bfloat16* __restrict__ w, void* __restrict__ out, int top, int N, int K, int unit,
+               const float* __restrict__ row_weights, float limit, float alpha) {
   extern __shared__ __align__(16) unsigned char few_smem[];
   __nv_bfloat16* rows = (__nv_bfloat16*)few_smem;            // FEW x K
   pdl_launch_dependents();
@@ -464,7 +475,7 @@ moe_few_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int* __r
   }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const bool gated = UP && limit > 0.f;               // else one matrix row per output
+  const bool gated = UP && unit != UNIT_PLAIN;        // else one matrix row per output
   const __nv_bfloat16* wexp = w + (size_t)e * (gated ? 2 * N : N) * K;
   for (int j = blockIdx.y * FEW_COLS + warp; j < min(N, (blockIdx.y + 1) * FEW_COLS); j += 8) {
     const __nv_bfloat16* w0 = wexp + (size_t)j * K;
@@ -502,9 +513,10 @@ moe_few_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int* __r
       const float g = warp_sum(s0[r]);
       if (UP) {
         const float u = gated ? warp_sum(s1[r]) : 0.f;
+        const float weight = row_weights ? row_weights[order[row0 + r]] : 1.0f;
         if (lane == 0)
           ((__nv_bfloat16*)out)[(size_t)(row0 + r) * N + j] = __float2bfloat16_rn(
-              glu(__bfloat162float(__float2bfloat16_rn(g)), __bfloat162float(__float2bfloat16_rn(u)), limit, alpha));
+              glu(unit, __bfloat162float(__float2bfloat16_rn(g * weight)), __bfloat162float(__float2bfloat16_rn(u * weight)), limit, alpha));
       } else if (lane == 0) {
         ((float*)out)[(size_t)(row0 + r) * N + j] = g;
       }
@@ -515,8 +527,8 @@ moe_few_kernel(const __nv_bfloat16* __restrict__ a, int a_stride, const int* __r
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(float* __restrict__ y, const T* __restrict__ h, int h_stride, const int* __restrict__ ids,
-                   const float* __restrict__ weights, const int* __restrict__ place_of, const float* __restrict__ rows,
-                   int width, int top) {
+                   const float* __restrict__ weights, float factor, const int* __restrict__ place_of,
+                   const float* __restrict__ rows, int width, int top) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -524,7 +536,7 @@ moe_combine_kernel(float* __restrict__ y, const T* __restrict__ h, int h_stride,
     float sum = 0.f;
     for (int place = 0; place < top; place++) {
       const int at = place_of[(size_t)t * top + place];
-      const float w = weights[(size_t)t * top + place];
+      const float w = weights ? weights[(size_t)t * top + place] : factor;
       sum = fmaf(w, at < 0 ? to_float(h[(size_t)t * h_stride + n]) : rows[(size_t)at * width + n], sum);
     }
     y[(size_t)t * width + n] += sum;
@@ -535,7 +547,7 @@ moe_combine_kernel(float* __restrict__ y, const T* __restrict__ h, int h_stride,
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_combine_vec_kernel(float* __restrict__ y, const T* __restrict__ h, int h_stride, const float* __restrict__ weights,
-                       const int* __restrict__ place_of, const float* __restrict__ rows, int width, int top) {
+                       float factor, const int* __restrict__ place_of, const float* __restrict__ rows, int width, int top) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -543,7 +555,7 @@ moe_combine_vec_kernel(float* __restrict__ y, const T* __restrict__ h, int h_str
     float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int place = 0; place < top; place++) {
       const int at = place_of[(size_t)t * top + place];
-      const float w = weights[(size_t)t * top + place];
+      const float w = weights ? weights[(size_t)t * top + place] : factor;
       float4 v;
       if (at < 0) {
         const T* src = h + (size_t)t * h_stride + n;
@@ -567,7 +579,7 @@ moe_combine_vec_kernel(float* __restrict__ y, const T* __restrict__ h, int h_str
 SPROUT_API int sprout_moe_route(const void* h, int h_stride, int dtype, const float* router, const float* correction, int* ids,
                                 float* weights, int* counts, int tokens, int width, int outputs, int experts, int top,
                                 float scale, int extra, float* extra_out, int group_count, int group_keep, int renormalize,
-                                cudaStream_t stream) {
+                                int sigmoid_scores, cudaStream_t stream) {
   SPROUT_REQUIRE(h && router && ids && weights && counts, "moe_route: null pointer");
   SPROUT_REQUIRE(extra >= 0 && (extra == 0 || extra_out), "moe_route: the extra rows' products need a place");
   SPROUT_REQUIRE(group_count >= 1 && group_keep >= 1 && group_keep <= group_count && outputs % group_count == 0,
@@ -591,7 +603,7 @@ SPROUT_API int sprout_moe_route(const void* h, int h_stride, int dtype, const fl
   dim3 grid((tokens + per_block - 1) / per_block);
 #define ROUTE(T, N)                                                                                                    \
   sprout_launch(moe_route_kernel<T, N>, grid, dim3(ROUTE_THREADS), smem, stream, (const T*)h, h_stride, router, correction, ids, \
-                weights, counts, tokens, width, outputs, experts, top, scale, extra, extra_out, group_count, group_keep, renormalize)
+                weights, counts, tokens, width, outputs, experts, top, scale, extra, extra_out, group_count, group_keep, renormalize, sigmoid_scores)
   if (dtype == SPROUT_F32) {
     if (per_block == 1) ROUTE(float, 1); else ROUTE(float, 8);
   } else if (dtype == SPROUT_BF16) {
@@ -614,18 +626,20 @@ SPROUT_API int sprout_moe_arrange(const int* ids, int* counts, int* offsets, int
 
 SPROUT_API int sprout_moe_up_plain(const void* h, int h_stride, int dtype, const int* sorted, const int* offsets,
                                    const void* w_gate_up, void* act, int max_rows, int experts, int top, int width, int ff,
-                                   float limit, float alpha, cudaStream_t stream) {
+                                   int unit, const float* row_weights, float limit, float alpha, cudaStream_t stream) {
   SPROUT_REQUIRE(h && sorted && offsets && w_gate_up && act && max_rows > 0 && experts > 0 && width > 0 && ff > 0,
                  "moe_up: bad arguments");
   SPROUT_REQUIRE(width <= 12000, "moe_up: width up to 12000");
+  SPROUT_REQUIRE(unit >= UNIT_CLAMPED && unit <= UNIT_SILU, "moe_up: unknown kind of expert %d", unit);
   dim3 grid(max_rows, ff >= 512 ? 4 : 1);
   const size_t smem = (size_t)width * sizeof(float);
   if (dtype == SPROUT_F32)
     sprout_launch(moe_up_plain_kernel<float>, grid, dim3(256), smem, stream, (const float*)h, h_stride, sorted, offsets,
-                  (const float*)w_gate_up, (float*)act, experts, top, width, ff, limit, alpha);
+                  (const float*)w_gate_up, (float*)act, experts, top, width, ff, unit, row_weights, limit, alpha);
   else if (dtype == SPROUT_BF16)
     sprout_launch(moe_up_plain_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)h, h_stride, sorted,
-                  offsets, (const __nv_bfloat16*)w_gate_up, (__nv_bfloat16*)act, experts, top, width, ff, limit, alpha);
+                  offsets, (const __nv_bfloat16*)w_gate_up, (__nv_bfloat16*)act, experts, top, width, ff, unit,
+                  row_weights, limit, alpha);
   else
     return sprout_fail("moe_up: unknown dtype %d", dtype);
   return sprout_check_launch("moe_up_plain");
@@ -657,8 +671,10 @@ SPROUT_API int sprout_moe_mma_supported(int width, int ff, int h_stride) {
 // act [entries, ff] bfloat16 = glu(W_gate a, W_up a); rows_out [entries, width] float32 = W_down act, over the arranged rows.
 SPROUT_API int sprout_moe_experts_mma(const void* h, int h_stride, const int* order, const int* offsets, const void* w_gate_up,
                                       const void* w_down, void* act, float* rows_out, int entries, int experts, int top,
-                                      int width, int ff, float limit, float alpha, cudaStream_t stream) {
+                                      int width, int ff, int unit, const float* row_weights, float limit, float alpha,
+                                      cudaStream_t stream) {
   SPROUT_REQUIRE(h && order && offsets && w_gate_up && w_down && act && rows_out, "moe_experts_mma: null pointer");
+  SPROUT_REQUIRE(unit >= UNIT_CLAMPED && unit <= UNIT_SILU, "moe_experts_mma: unknown kind of expert %d", unit);
   SPROUT_REQUIRE(entries > 0 && experts > 0 && top > 0 && sprout_moe_mma_supported(width, ff, h_stride),
                  "moe_experts_mma: sizes must be multiples of 8 (width %d, ff %d, row stride %d)", width, ff, h_stride);
   SPROUT_REQUIRE((((uintptr_t)h | (uintptr_t)w_gate_up | (uintptr_t)w_down | (uintptr_t)act | (uintptr_t)rows_out) & 15) == 0,
@@ -672,10 +688,12 @@ SPROUT_API int sprout_moe_experts_mma(const void* h, int h_stride, const int* or
       few_prepared = true;
     }
     sprout_launch(moe_few_kernel<true>, dim3(experts, (ff + FEW_COLS - 1) / FEW_COLS), dim3(256), (size_t)FEW * width * 2, stream,
-                  (const __nv_bfloat16*)h, h_stride, order, offsets, (const __nv_bfloat16*)w_gate_up, act, top, ff, width, limit, alpha);
+                  (const __nv_bfloat16*)h, h_stride, order, offsets, (const __nv_bfloat16*)w_gate_up, act, top, ff, width, unit, row_weights,
+                  limit, alpha);
     if (int code = sprout_check_launch("moe_up_few")) return code;
     sprout_launch(moe_few_kernel<false>, dim3(experts, (width + FEW_COLS - 1) / FEW_COLS), dim3(256), (size_t)FEW * ff * 2, stream,
-                  (const __nv_bfloat16*)act, ff, order, offsets, (const __nv_bfloat16*)w_down, (void*)rows_out, top, width, ff, 0.f, 0.f);
+                  (const __nv_bfloat16*)act, ff, order, offsets, (const __nv_bfloat16*)w_down, (void*)rows_out, top, width, ff, unit,
+                  (const float*)nullptr, 0.f, 0.f);
     return sprout_check_launch("moe_down_few");
   }
   static bool prepared = false;
@@ -686,38 +704,38 @@ SPROUT_API int sprout_moe_experts_mma(const void* h, int h_stride, const int* or
     prepared = true;
   }
   const int tiles = (entries + GM - 1) / GM + experts;       // at most this many row tiles, whatever the routing
-  if (limit > 0.f)
+  if (unit != UNIT_PLAIN)
     sprout_launch(moe_gemm_mma_kernel<1>, dim3(tiles, (ff + GN / 2 - 1) / (GN / 2)), dim3(GTHREADS), GEMM_SMEM, stream,
                   (const __nv_bfloat16*)h, h_stride, order, offsets, (const __nv_bfloat16*)w_gate_up, act, experts, top, ff, width,
-                  limit, alpha);
+                  unit, row_weights, limit, alpha);
   else
     sprout_launch(moe_gemm_mma_kernel<2>, dim3(tiles, (ff + GN - 1) / GN), dim3(GTHREADS), GEMM_SMEM, stream,
                   (const __nv_bfloat16*)h, h_stride, order, offsets, (const __nv_bfloat16*)w_gate_up, act, experts, top, ff, width,
-                  limit, alpha);
+                  unit, row_weights, limit, alpha);
   if (int code = sprout_check_launch("moe_up_mma")) return code;
   sprout_launch(moe_gemm_mma_kernel<0>, dim3(tiles, (width + GN - 1) / GN), dim3(GTHREADS), GEMM_SMEM, stream,
                 (const __nv_bfloat16*)act, ff, order, offsets, (const __nv_bfloat16*)w_down, (void*)rows_out, experts, top, width, ff,
-                0.f, 0.f);
+                unit, (const float*)nullptr, 0.f, 0.f);
   return sprout_check_launch("moe_down_mma");
 }
 
 SPROUT_API int sprout_moe_combine(float* y, const void* h, int h_stride, int dtype, const int* ids, const float* weights,
-                                  const int* place_of, const float* rows, int tokens, int width, int top,
+                                  float factor, const int* place_of, const float* rows, int tokens, int width, int top,
                                   cudaStream_t stream) {
-  SPROUT_REQUIRE(y && h && ids && weights && place_of && tokens > 0 && width > 0 && top > 0, "moe_combine: bad arguments");
+  SPROUT_REQUIRE(y && h && ids && place_of && tokens > 0 && width > 0 && top > 0, "moe_combine: bad arguments");
   const bool vec = width % 4 == 0 && (((uintptr_t)y | (uintptr_t)rows) & 15) == 0;
   if (vec && dtype == SPROUT_F32)
-    sprout_launch(moe_combine_vec_kernel<float>, dim3(tokens), dim3(256), 0, stream, y, (const float*)h, h_stride, weights, place_of,
+    sprout_launch(moe_combine_vec_kernel<float>, dim3(tokens), dim3(256), 0, stream, y, (const float*)h, h_stride, weights, factor, place_of,
                   rows, width, top);
   else if (vec && dtype == SPROUT_BF16)
     sprout_launch(moe_combine_vec_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, y, (const __nv_bfloat16*)h, h_stride,
-                  weights, place_of, rows, width, top);
+                  weights, factor, place_of, rows, width, top);
   else if (dtype == SPROUT_F32)
     sprout_launch(moe_combine_kernel<float>, dim3(tokens), dim3(256), 0, stream, y, (const float*)h, h_stride, ids, weights,
-                  place_of, rows, width, top);
+                  factor, place_of, rows, width, top);
   else if (dtype == SPROUT_BF16)
     sprout_launch(moe_combine_kernel<__nv_bfloat16>, dim3(tokens), dim3(256), 0, stream, y, (const __nv_bfloat16*)h, h_stride,
-                  ids, weights, place_of, rows, width, top);
+                  ids, weights, factor, place_of, rows, width, top);
   else
     return sprout_fail("moe_combine: unknown dtype %d", dtype);
   return sprout_check_launch("moe_combine");

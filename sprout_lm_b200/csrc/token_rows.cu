@@ -8,6 +8,8 @@
 //  * side_gate:      out[t, j] = gelu_tanh(z[t, j]) * table[token[t], first + j]: a per-token row of a table gated by a
 //                    projection of the stream.
 //  * rms_add:        x[t] += y[t] / sqrt(mean(y[t]^2) + eps) * w: a normed row added to the stream.
+//  * rms_pair_add:   x[t] += factor * (y1[t] / rms(y1[t]) * w1 + y2[t] / rms(y2[t]) * w2): two sublayers' outputs, each normed
+//                    over the stream's width, weighed alike and added.
 //  * add_rows:       x[t] += vec (+ other[t]): a learned vector, and optionally another stream, added to every row.
 //  * gated_rows_add: x[t] += sigmoid(logit[t]) * y[t]: a sublayer's float32 rows weighed by one number per token.
 //  * narrow_rows:    the float32 stream in bfloat16, for a product that reads the stream itself.
@@ -88,6 +90,25 @@ side_gate_kernel(const T* __restrict__ z, int z_stride, const T* __restrict__ ta
 }
 
 // a block per row
+__global__ void __launch_bounds__(256)
+rms_pair_add_kernel(const float* __restrict__ y1, const float* __restrict__ y2, const float* __restrict__ w1,
+                    const float* __restrict__ w2, float* __restrict__ x, int width, float eps, float factor) {
+  __shared__ float scratch[33];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t at = (size_t)blockIdx.x * width;
+  float q1 = 0.f, q2 = 0.f;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float a = y1[at + i], b = y2[at + i];
+    q1 = fmaf(a, a, q1);
+    q2 = fmaf(b, b, q2);
+  }
+  const float r1 = factor / sqrtf(block_sum(q1, scratch) / (float)width + eps);
+  const float r2 = factor / sqrtf(block_sum(q2, scratch) / (float)width + eps);
+  for (int i = threadIdx.x; i < width; i += blockDim.x)
+    x[at + i] += y1[at + i] * r1 * w1[i] + y2[at + i] * r2 * w2[i];
+}
+
 __global__ void __launch_bounds__(256)
 rms_add_kernel(const float* __restrict__ y, const float* __restrict__ weight, float* __restrict__ x, int width, float eps) {
   __shared__ float scratch[33];
@@ -293,6 +314,13 @@ SPROUT_API int sprout_rms_add(const float* y, const float* weight, float* x, int
   SPROUT_REQUIRE(y && weight && x && rows > 0 && width > 0 && eps > 0.f, "rms_add: bad arguments");
   sprout_launch(rms_add_kernel, dim3(rows), dim3(256), 0, stream, y, weight, x, width, eps);
   return sprout_check_launch("rms_add");
+}
+
+SPROUT_API int sprout_rms_pair_add(const float* y1, const float* y2, const float* w1, const float* w2, float* x, int rows, int width,
+                                   float eps, float factor, cudaStream_t stream) {
+  SPROUT_REQUIRE(y1 && y2 && w1 && w2 && x && rows > 0 && width > 0 && eps > 0.f, "rms_pair_add: bad arguments");
+  sprout_launch(rms_pair_add_kernel, dim3(rows), dim3(256), 0, stream, y1, y2, w1, w2, x, width, eps, factor);
+  return sprout_check_launch("rms_pair_add");
 }
 
 SPROUT_API int sprout_add_rows(float* x, const float* other, const float* vec, int rows, int width, cudaStream_t stream) {

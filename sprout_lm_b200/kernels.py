@@ -30,6 +30,7 @@ class KernelError(RuntimeError):
 _P, _I, _F, _L = c_void_p, c_int, c_float, ctypes.c_longlong
 _SIGNATURES = {
     "sprout_embed": [_P, _I, _P, _P, _I, _I, _I, _F, _P, _P],
+    "sprout_embed_pairs": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _F, _L, _L, _I, _P, _P],
     "sprout_rmsnorm": [_P, _P, _P, _I, _P, _I, _I, _F, _P],
     "sprout_swiglu": [_P, _P, _I, _I, _I, _I, _P],
     "sprout_rope_append": [_P, _P, _P, _I, _P, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
@@ -67,34 +68,38 @@ _SIGNATURES = {
     "sprout_gated_rmsnorm": [_P, _P, _P, _I, _P, _I, _I, _I, _F, _P],
     "sprout_relu2": [_P, _P, _I, _L, _P],
     "sprout_glu_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
-    "sprout_rope_maps_append": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _F, _P, _P],
-    "sprout_multimap_attention_simple": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _I, _P, _P, _I, _I, _F, _P, _P],
-    "sprout_multimap_attention_mma": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _P, _I, _I, _P, _P, _I, _I, _F, _P, _P],
+    "sprout_rope_maps_append": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _F, _I, _I, _P, _P, _P, _P],
+    "sprout_multimap_attention_simple": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _I, _P, _P, _I, _I, _F,
+                                         _I, _P, _P, _I, _I, _P, _P],
+    "sprout_multimap_attention_mma": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _P, _I, _I, _P, _P, _I, _I, _F,
+                                      _I, _P, _P, _I, _I, _P, _P],
     "sprout_multimap_attention_mma_supported": [_I, _I, _I],
     "sprout_decay_chunks": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "sprout_decay_chunks_supported": [_I, _I, _I],
     "sprout_decay_scan": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "sprout_gated_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _P, _P, _P, _F, _F, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P,
-                          _I, _I, _I, _P, _P, _P, _P, _I, _I, _P],
+                          _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P],
+    "sprout_delta_rule": [_P, _P, _P, _I, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _P, _P, _I, _P, _I, _P, _P, _P],
     "sprout_causal_conv": [_P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "sprout_gated_group_norm": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _F, _I, _I, _P],
     "sprout_scaled_sum": [_P, _P, _F, _P, _F, _L, _P],
-    "sprout_moe_route": [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _I, _I, _P],
+    "sprout_moe_route": [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _I, _I, _I, _P],
     "sprout_exp_gates": [_P, _P, _I, _P, _P, _F, _I, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P],
     "sprout_exp_memory_out": [_P, _I, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P],
     "sprout_unit_act": [_P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "sprout_side_input_few": [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _P],
     "sprout_side_gate": [_P, _I, _P, _I, _I, _P, _I, _P, _I, _I, _I, _P, _P],
     "sprout_rms_add": [_P, _P, _P, _I, _I, _F, _P],
+    "sprout_rms_pair_add": [_P, _P, _P, _P, _P, _I, _I, _F, _F, _P],
     "sprout_add_rows": [_P, _P, _P, _I, _I, _P],
     "sprout_gated_rows_add": [_P, _P, _P, _I, _I, _I, _P],
     "sprout_narrow_rows": [_P, _P, _L, _P],
     "sprout_moe_arrange": [_P, _P, _P, _P, _P, _I, _I, _P],
-    "sprout_moe_up_plain": [_P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
+    "sprout_moe_up_plain": [_P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _F, _F, _P],
     "sprout_moe_down_plain": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _P],
-    "sprout_moe_combine": [_P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P],
+    "sprout_moe_combine": [_P, _P, _I, _I, _P, _P, _F, _P, _P, _I, _I, _I, _P],
     "sprout_moe_mma_supported": [_I, _I, _I],
-    "sprout_moe_experts_mma": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
+    "sprout_moe_experts_mma": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _F, _F, _P],
 }
 
 _lock = threading.Lock()
@@ -113,6 +118,8 @@ def load_library(verbose: bool = True):
             lib.sprout_abi_version.restype = c_int
             lib.sprout_sample_scratch_bytes.restype = ctypes.c_longlong
             lib.sprout_sample_scratch_bytes.argtypes = [c_int]
+            lib.sprout_delta_scratch_floats.restype = ctypes.c_longlong
+            lib.sprout_delta_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
             lib.sprout_attention_decode_scratch_floats.restype = ctypes.c_longlong
             lib.sprout_attention_decode_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
             lib.sprout_attention_decode_ctas_per_sm.restype = c_int
@@ -213,6 +220,24 @@ def embed(table, tokens, out, status, scale: float = 1.0):
         raise KernelError("embed: shapes do not fit")
     _run("sprout_embed", _ptr(table, "table"), _dtype_code(table.dtype), _ptr(tokens, "tokens", torch.int32),
          _ptr(out, "out", torch.float32), T, H, table.shape[0], float(scale), _ptr(status, "status", torch.int32), _stream())
+
+
+def embed_pairs(table, pairs, ctx, state, out, scale: float, mul_prev: int, mul_cur: int, status):
+    """out[t] = table[token] * scale + pairs[(previous token * mul_prev + token * mul_cur) mod (rows - 1)], float32; a sequence's
+    first token takes the last row of ``pairs``.  ``state`` (int32 [slots, 1]): each request's last token, read for the first
+    token it brings and brought up to date."""
+    T, H = out.shape
+    buffer = state.buffer
+    if not table.is_contiguous() or not pairs.is_contiguous() or not out.is_contiguous() or table.dtype != pairs.dtype \
+            or table.shape[1] != H or pairs.shape[1] != H or pairs.shape[0] < 2 or ctx.token_ids.numel() != T:
+        raise KernelError("embed_pairs: shapes or dtypes do not fit")
+    if buffer.dtype != torch.int32 or not buffer.is_contiguous() or buffer.numel() != buffer.shape[0]:
+        raise KernelError("embed_pairs: the last tokens are contiguous int32, one per slot")
+    _run("sprout_embed_pairs", _ptr(table, "table"), _ptr(pairs, "pairs"), _dtype_code(table.dtype), _ptr(ctx.token_ids, "tokens", torch.int32),
+         _ptr(ctx.positions, "positions", torch.int32), _ptr(ctx.seq_of_token, "seq_of_token", torch.int32),
+         _ptr(ctx.q_start, "q_start", torch.int32), _ptr(state.slots, "state_slots", torch.int32), _ptr(buffer, "last_token", torch.int32),
+         buffer.shape[0], _ptr(out, "out", torch.float32), T, H, table.shape[0], float(scale), int(mul_prev), int(mul_cur),
+         pairs.shape[0] - 1, _ptr(status, "status", torch.int32), _stream())
 
 
 def rmsnorm(x, gain, out, eps, rows=None):
@@ -1166,22 +1191,33 @@ def glu_clamped(gate_up, out, limit: float, alpha: float):
 
 def rope_maps_append(rows, positions, seq_of_token, block_table, cos_table, sin_table, k_cache, v_cache, q_vectors: int,
                      kv_heads: int, maps: int, dim: int, vdim: int, page_tokens: int, write: bool, status,
-                     unit_eps: float = 0.0, value_from_key: bool = False, q_weight=None, k_weight=None, weight_eps: float = 0.0):
+                     unit_eps: float = 0.0, value_from_key: bool = False, q_weight=None, k_weight=None, weight_eps: float = 0.0,
+                     interleaved: bool = False, value_turn=None):
     """Rotate the first ``2 * cos_table.shape[1]`` elements of every query vector (in place) and key vector by the token's
-    position, half-split pairs; append keys ([pages, kv_heads, page_tokens, maps * dim]) and values
+    position, in half-split pairs or, with ``interleaved``, in pairs (2i, 2i + 1); append keys ([pages, kv_heads, page_tokens, maps * dim]) and values
     ([pages, kv_heads, page_tokens, vdim]) when ``write``.  A row holds q_vectors * dim query elements, then (when
     ``write``) kv_heads * maps * dim key elements and kv_heads * vdim value elements.  With ``unit_eps`` > 0 every query
     and key vector is divided by its root mean square over ``dim`` after the rotation; with ``value_from_key`` the rows hold
     no value elements and the cached value row is the key row as projected (before rotation and norm).  ``q_weight`` /
     ``k_weight`` (float32 [dim]): before the rotation every query / key vector is divided by its root mean square over
-    ``dim`` (``weight_eps`` inside the root) and multiplied by the weight."""
+    ``dim`` (``weight_eps`` inside the root) and multiplied by the weight; weights as wide as all query vectors and all key
+    vectors together ([q_vectors * dim] and [kv_heads * maps * dim]): the norm is over the token's whole projection instead.
+    ``value_turn`` = (cos, sin), tables [max_positions, vdim / 2]: value rows are turned by the token's position over all of
+    their elements before they are cached, in pairs like the keys'."""
     _rows_contiguous(rows, "rows")
+    weights = [(w, width) for w, width in ((q_weight, q_vectors * dim), (k_weight, kv_heads * maps * dim)) if w is not None]
+    whole = all(w.numel() == width for w, width in weights) and any(w.numel() != dim for w, _ in weights)
     for weight in (q_weight, k_weight):
-        if weight is not None and (weight.dtype != torch.float32 or weight.numel() != dim or not weight.is_contiguous()):
-            raise KernelError("rope_maps_append: a norm weight is float32 [dim]")
+        if weight is not None and (weight.dtype != torch.float32 or (not whole and weight.numel() != dim) or not weight.is_contiguous()):
+            raise KernelError("rope_maps_append: a norm weight is float32 [dim], or as wide as the whole projection")
     _rows_contiguous(block_table, "block_table")
     T = rows.shape[0]
     cos_ptr, sin_ptr, max_positions, rot = _rotary(cos_table, sin_table, dim, "rope_maps_append")
+    v_cos, v_sin, turned = _turn_args(value_turn, vdim, "rope_maps_append")
+    if v_cos is not None:
+        if rot and max_positions != turned:
+            raise KernelError("rope_maps_append: the keys' and the values' tables cover different positions")
+        max_positions = turned
     if write:
         if k_cache.dtype != rows.dtype or not k_cache.is_contiguous() or tuple(k_cache.shape[1:]) != (kv_heads, page_tokens, maps * dim):
             raise KernelError("rope_maps_append: k_cache must be contiguous [pages, kv_heads, page_tokens, maps * dim]")
@@ -1193,7 +1229,8 @@ def rope_maps_append(rows, positions, seq_of_token, block_table, cos_table, sin_
          _ptr(k_cache, "k_cache", allow_none=not write), _ptr(v_cache, "v_cache", allow_none=not write), T, q_vectors,
          kv_heads, maps, dim, rot, vdim, page_tokens, k_cache.shape[0] if write else 1, 1 if write else 0,
          float(unit_eps), 1 if value_from_key else 0, _ptr(q_weight, "q_weight", torch.float32, True),
-         _ptr(k_weight, "k_weight", torch.float32, True), float(weight_eps), _ptr(status, "status", torch.int32), _stream())
+         _ptr(k_weight, "k_weight", torch.float32, True), float(weight_eps), 1 if whole else 0, 1 if interleaved else 0, v_cos, v_sin,
+         _ptr(status, "status", torch.int32), _stream())
 
 
 MASK_KINDS = {"causal": 0, "window": 1, "chunk": 2}
@@ -1213,25 +1250,39 @@ def _mask_code(mask) -> tuple[int, int, int]:
     return MASK_KINDS[kind], int(size or 0), keep
 
 
-def _gate_args(gate, tokens: int, heads: int, dtype, name: str):
+def _gate_args(gate, tokens: int, heads: int, vdim: int, dtype, name: str):
+    """(pointer, row stride, whether the gate has a number per element of the output instead of one per head)."""
     if gate is None:
-        return None, 0
-    if gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] != tokens or gate.shape[1] != heads or gate.dtype != dtype:
-        raise KernelError(f"{name}: the gate must be a [tokens, heads] view with unit inner stride, of q's dtype")
-    return gate.data_ptr(), gate.stride(0)
+        return None, 0, 0
+    if gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[0] != tokens or gate.shape[1] not in (heads, heads * vdim) or gate.dtype != dtype:
+        raise KernelError(f"{name}: the gate must be a [tokens, heads] or [tokens, heads * vdim] view with unit inner stride, of q's dtype")
+    return gate.data_ptr(), gate.stride(0), 0 if gate.shape[1] == heads else 1
+
+
+def _turn_args(turn, vdim: int, name: str):
+    """(cos pointer, sin pointer, positions) of tables [positions, vdim / 2], or (None, None, 0)."""
+    if turn is None:
+        return None, None, 0
+    cos, sin = turn[0], turn[1]
+    if cos.shape != sin.shape or cos.dim() != 2 or 2 * cos.shape[1] != vdim or not cos.is_contiguous() or not sin.is_contiguous():
+        raise KernelError(f"{name}: the values' tables must be contiguous [positions, vdim / 2]")
+    return _ptr(cos, "cos", torch.float32), _ptr(sin, "sin", torch.float32), cos.shape[0]
 
 
 def multimap_attention_simple(q, cache, ctx, out, heads: int, kv_heads: int, maps: int, dim: int, vdim: int, scale: float,
                               lam: float, norm_eps: float, out_scale: float, status, mask=None, sink=None, gate=None,
-                              softcap: float = 0.0):
+                              softcap: float = 0.0, turn=None, interleaved: bool = False):
     """Causal attention with ``maps`` (1 or 2) softmax maps per head over shared values, float32 arithmetic:
     out = (a_0 - lam a_1) [/ rms when norm_eps > 0] * out_scale per head.  q [tokens, heads * maps * dim] (a view with
     unit inner stride), out [tokens, heads * vdim].  ``mask`` says what a query sees (``_mask_code``), ``sink`` (float32
     [heads]) adds exp(sink_h) to every softmax denominator of head h, ``gate`` ([tokens, heads]) multiplies head h's output
-    by sigmoid(gate); ``softcap`` > 0 turns every scaled score s into softcap * tanh(s / softcap)."""
+    by sigmoid(gate), or with [tokens, heads * vdim] every element by its own; ``softcap`` > 0 turns every scaled score s into
+    softcap * tanh(s / softcap); ``turn`` = (cos, sin), tables [positions, vdim / 2]: a head's output is turned back by the
+    query's position before the gate (pairs (2i, 2i + 1) with ``interleaved``, else half-split)."""
     _rows_contiguous(q, "q")
     mask_kind, mask_size, mask_keep = _mask_code(mask)
-    gate_ptr, gate_stride = _gate_args(gate, q.shape[0], heads, q.dtype, "multimap_attention")
+    gate_ptr, gate_stride, gate_elements = _gate_args(gate, q.shape[0], heads, vdim, q.dtype, "multimap_attention")
+    turn_cos, turn_sin, turned = _turn_args(turn, vdim, "multimap_attention")
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != heads):
         raise KernelError("multimap_attention: one float32 sink per head")
     _rows_contiguous(out, "out")
@@ -1247,8 +1298,8 @@ def multimap_attention_simple(q, cache, ctx, out, heads: int, kv_heads: int, map
          _ptr(ctx.seq_of_token, "seq_of_token", torch.int32), _ptr(ctx.positions, "positions", torch.int32), _ptr(out, "out"),
          out.stride(0), _dtype_code(q.dtype), q.shape[0], heads, kv_heads, maps, dim, vdim, cache.page_tokens,
          k_cache.shape[0], float(scale), float(lam), float(norm_eps), float(out_scale), mask_kind, mask_size,
-         _ptr(sink, "sink", torch.float32, True), gate_ptr, gate_stride, mask_keep, float(softcap),
-         _ptr(status, "status", torch.int32), _stream())
+         _ptr(sink, "sink", torch.float32, True), gate_ptr, gate_stride, mask_keep, float(softcap), gate_elements,
+         turn_cos, turn_sin, turned, 1 if interleaved else 0, _ptr(status, "status", torch.int32), _stream())
 
 
 # ---------------------------------------------------------------------------------- linear attention with decay and state
@@ -1271,10 +1322,11 @@ def decay_scan(rows, q_start, state_slots, state, decay, out, heads: int, dim: i
 # ---------------------------------------------------------------------------------- routed feed-forward
 
 def moe_route(h, router, correction, ids, weights, counts, experts: int, top: int, scale: float, groups=None,
-              renormalize: bool = True, extra_out=None):
+              renormalize: bool = True, extra_out=None, sigmoid: bool = False):
     """Per token: softmax of the float32 router product, ``top`` largest of score + correction (lowest index first among
     equals; ``correction`` None: the scores alone), weights = taken scores / (their sum + 1e-20) * scale, or the taken
-    scores * scale when not ``renormalize``.  ``groups`` = (count, keep): the outputs form ``count`` equal groups of
+    scores * scale when not ``renormalize``.  ``sigmoid``: the scores are the sigmoids of the single products instead of their
+    softmax.  ``groups`` = (count, keep): the outputs form ``count`` equal groups of
     neighbours, a group's score is its largest score, only outputs of the ``keep`` best groups can be taken.  ``extra_out``
     (float32 [tokens, n]): the router matrix's last n rows are not part of the softmax; their products are written there.
     ids int32 [tokens, top] (from ``experts`` on: identity experts), weights float32 [tokens, top]; counts int32 [experts] +=
@@ -1292,7 +1344,8 @@ def moe_route(h, router, correction, ids, weights, counts, experts: int, top: in
     _run("sprout_moe_route", _ptr(h, "h"), h.stride(0), _dtype_code(h.dtype), _ptr(router, "router", torch.float32),
          _ptr(correction, "correction", torch.float32, True), _ptr(ids, "ids", torch.int32), _ptr(weights, "weights", torch.float32),
          _ptr(counts, "counts", torch.int32), T, width, outputs, experts, top, float(scale), extra,
-         _ptr(extra_out, "extra_out", torch.float32, True), group_count, group_keep, 1 if renormalize else 0, _stream())
+         _ptr(extra_out, "extra_out", torch.float32, True), group_count, group_keep, 1 if renormalize else 0,
+         1 if sigmoid else 0, _stream())
 
 
 def moe_arrange(ids, counts, offsets, order, place_of, experts: int):
@@ -1306,18 +1359,38 @@ def moe_arrange(ids, counts, offsets, order, place_of, experts: int):
          entries, experts, _stream())
 
 
-def moe_up_plain(h, order, offsets, w_gate_up, act, experts: int, top: int, limit: float, alpha: float):
+EXPERT_UNITS = {"clamped_glu": 0, "plain": 1, "silu_glu": 2}
+
+
+def _unit_code(unit, limit: float) -> int:
+    if unit is None:
+        return EXPERT_UNITS["clamped_glu" if limit > 0 else "plain"]
+    if unit not in EXPERT_UNITS:
+        raise KernelError(f"unknown kind of expert {unit!r}")
+    return EXPERT_UNITS[unit]
+
+
+def _row_weights_ptr(row_weights, entries: int):
+    if row_weights is not None and (row_weights.numel() != entries or not row_weights.is_contiguous()):
+        raise KernelError("experts: one float32 weight per token and place")
+    return _ptr(row_weights, "row_weights", torch.float32, True)
+
+
+def moe_up_plain(h, order, offsets, w_gate_up, act, experts: int, top: int, limit: float, alpha: float, unit=None, row_weights=None):
     """act[row] = glu_clamped(W_gate[e] a, W_up[e] a) for the arranged rows (a = h[order[row] // top], e the row's expert);
     w_gate_up [experts, 2 ff, width] with gate rows first; CUDA cores, float32 sums in ascending k.  ``limit`` <= 0: experts
-    without a gate, act[row] = gelu(W_up[e] a) (the exact form) with w_gate_up [experts, ff, width]."""
+    without a gate, act[row] = gelu(W_up[e] a) (the exact form) with w_gate_up [experts, ff, width].  ``unit`` names the kind
+    of expert where the limit does not: "silu_glu" is silu(W_gate a) * (W_up a).  ``row_weights`` (float32 [tokens, top])
+    multiply an expert's input, a = weight * h[order[row] // top]."""
     _rows_contiguous(h, "h")
     R, ff = act.shape
-    if not w_gate_up.is_contiguous() or tuple(w_gate_up.shape) != (experts, (2 if limit > 0 else 1) * ff, h.shape[1]) or w_gate_up.dtype != h.dtype \
+    code = _unit_code(unit, limit)
+    if not w_gate_up.is_contiguous() or tuple(w_gate_up.shape) != (experts, (1 if code == EXPERT_UNITS["plain"] else 2) * ff, h.shape[1]) or w_gate_up.dtype != h.dtype \
             or act.dtype != h.dtype or not act.is_contiguous():
         raise KernelError("moe_up: shapes or dtypes do not fit")
     _run("sprout_moe_up_plain", _ptr(h, "h"), h.stride(0), _dtype_code(h.dtype), _ptr(order, "order", torch.int32),
          _ptr(offsets, "offsets", torch.int32), _ptr(w_gate_up, "w_gate_up"), _ptr(act, "act"), R, experts, top, h.shape[1], ff,
-         float(limit), float(alpha), _stream())
+         code, _row_weights_ptr(row_weights, R), float(limit), float(alpha), _stream())
 
 
 def moe_down_plain(act, offsets, w_down, rows_out, experts: int):
@@ -1331,14 +1404,15 @@ def moe_down_plain(act, offsets, w_down, rows_out, experts: int):
          _ptr(w_down, "w_down"), _ptr(rows_out, "rows_out", torch.float32), R, experts, width, ff, _stream())
 
 
-def moe_combine(y, h, ids, weights, place_of, rows, top: int):
-    """y[t] += sum over the token's places of weight * (h[t] for an identity expert, else rows[place_of])."""
+def moe_combine(y, h, ids, weights, place_of, rows, top: int, factor: float = 1.0):
+    """y[t] += sum over the token's places of weight * (h[t] for an identity expert, else rows[place_of]); with ``weights``
+    None every place has the weight ``factor``."""
     _rows_contiguous(h, "h")
     T, width = y.shape
     if not y.is_contiguous() or y.dtype != torch.float32 or h.shape != y.shape or (rows is not None and rows.shape[1] != width):
         raise KernelError("moe_combine: shapes do not fit")
     _run("sprout_moe_combine", _ptr(y, "y", torch.float32), _ptr(h, "h"), h.stride(0), _dtype_code(h.dtype),
-         _ptr(ids, "ids", torch.int32), _ptr(weights, "weights", torch.float32), _ptr(place_of, "place_of", torch.int32),
+         _ptr(ids, "ids", torch.int32), _ptr(weights, "weights", torch.float32, True), float(factor), _ptr(place_of, "place_of", torch.int32),
          _ptr(rows, "rows", torch.float32, True), T, width, top, _stream())
 
 
@@ -1360,7 +1434,8 @@ def visible_keys(mask, context: int) -> int:
 
 
 def multimap_attention(q, cache, ctx, out, heads: int, kv_heads: int, maps: int, dim: int, vdim: int, scale: float, lam: float,
-                       norm_eps: float, out_scale: float, status, mask=None, sink=None, gate=None, softcap: float = 0.0):
+                       norm_eps: float, out_scale: float, status, mask=None, sink=None, gate=None, softcap: float = 0.0, turn=None,
+                       interleaved: bool = False):
     """Attention with one or two maps per head: the tensor-core kernel in bfloat16 for the sizes it is built for
     (``SPROUT_MULTIMAP_ATTENTION=simple`` keeps the float32-arithmetic kernel), else the float32-arithmetic kernel."""
     if q.dtype == torch.bfloat16 and os.environ.get("SPROUT_MULTIMAP_ATTENTION", "mma") != "simple" \
@@ -1382,7 +1457,8 @@ def multimap_attention(q, cache, ctx, out, heads: int, kv_heads: int, maps: int,
         planned = int(getattr(ctx, "planned_context", 0) or getattr(ctx, "max_context", 0) or 0)
         ksplit = multimap_key_split(requests, kv_heads, group, max_q_len, visible_keys(mask, planned)) if planned else 1
         mask_kind, mask_size, mask_keep = _mask_code(mask)
-        gate_ptr, gate_stride = _gate_args(gate, q.shape[0], heads, q.dtype, "multimap_attention")
+        gate_ptr, gate_stride, gate_elements = _gate_args(gate, q.shape[0], heads, vdim, q.dtype, "multimap_attention")
+        turn_cos, turn_sin, turned = _turn_args(turn, vdim, "multimap_attention")
         if sink is not None and (sink.dtype != torch.float32 or sink.numel() != heads):
             raise KernelError("multimap_attention: one float32 sink per head")
         partial = None
@@ -1396,10 +1472,10 @@ def multimap_attention(q, cache, ctx, out, heads: int, kv_heads: int, maps: int,
              cache.page_tokens, k_cache.shape[0], float(scale),
              float(lam), float(norm_eps), float(out_scale), ksplit, _ptr(partial, "partial", torch.float32, True),
              mask_kind, mask_size, _ptr(sink, "sink", torch.float32, True), gate_ptr, gate_stride, mask_keep, float(softcap),
-             _ptr(status, "status", torch.int32), _stream())
+             gate_elements, turn_cos, turn_sin, turned, 1 if interleaved else 0, _ptr(status, "status", torch.int32), _stream())
         return
     multimap_attention_simple(q, cache, ctx, out, heads, kv_heads, maps, dim, vdim, scale, lam, norm_eps, out_scale, status,
-                              mask=mask, sink=sink, gate=gate, softcap=softcap)
+                              mask=mask, sink=sink, gate=gate, softcap=softcap, turn=turn, interleaved=interleaved)
 
 
 CHUNKED_FROM = 8            # a step whose longest portion has at least this many tokens runs the chunked decay kernel
@@ -1439,8 +1515,9 @@ def decay_attention(rows, ctx, state, decay, out, heads: int, dim: int, vdim: in
     decay_scan(rows, ctx.q_start, state.slots, state.buffer, decay, out, heads, dim, vdim, silu, status)
 
 
-def moe_experts(h, order, offsets, w_gate_up, w_down, act, rows_out, experts: int, top: int, limit: float, alpha: float):
-    """The routed experts' two products over the arranged rows: on tensor cores in bfloat16 when the sizes are
+def moe_experts(h, order, offsets, w_gate_up, w_down, act, rows_out, experts: int, top: int, limit: float, alpha: float, unit=None,
+                row_weights=None):
+    """The routed experts' two products over the arranged rows (``unit``, ``row_weights``: see ``moe_up_plain``): on tensor cores in bfloat16 when the sizes are
     multiples of 8 (``SPROUT_MOE=plain`` keeps the CUDA-core products), else on CUDA cores."""
     global LAUNCHES
     width, ff = h.shape[1], act.shape[1]
@@ -1450,10 +1527,11 @@ def moe_experts(h, order, offsets, w_gate_up, w_down, act, rows_out, experts: in
         _run("sprout_moe_experts_mma", _ptr(h, "h"), h.stride(0), _ptr(order, "order", torch.int32),
              _ptr(offsets, "offsets", torch.int32), _ptr(w_gate_up, "w_gate_up", torch.bfloat16),
              _ptr(w_down, "w_down", torch.bfloat16), _ptr(act, "act", torch.bfloat16), _ptr(rows_out, "rows_out", torch.float32),
-             act.shape[0], experts, top, width, ff, float(limit), float(alpha), _stream())
+             act.shape[0], experts, top, width, ff, _unit_code(unit, limit), _row_weights_ptr(row_weights, act.shape[0]), float(limit),
+             float(alpha), _stream())
         LAUNCHES += 1               # two kernels behind one call
         return
-    moe_up_plain(h, order, offsets, w_gate_up, act, experts, top, limit, alpha)
+    moe_up_plain(h, order, offsets, w_gate_up, act, experts, top, limit, alpha, unit=unit, row_weights=row_weights)
     moe_down_plain(act, offsets, w_down, rows_out, experts)
 
 
@@ -1471,12 +1549,15 @@ def _scan_view(t, name: str, width: int, dtype):
 
 
 def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: int, vdim: int, status, per_head: bool = False,
-               tau: float = 1.0, q_scale: float = 1.0, a_log=None, skip=None, given=None, ones_col: bool = False):
+               tau: float = 1.0, q_scale: float = 1.0, a_log=None, skip=None, given=None, ones_col: bool = False, floor=None,
+               q_silu: bool = False):
     """Per request and head, token by token: S = diag(a) S + (c k) v^T, o = S^T (q_scale q) + skip_h v, the state float32
     [slots, heads, dim, vdim] read and written at the requests' slots (``state``: a ``StateView``-like with ``buffer`` and
     ``slots``).  q, k [tokens, groups * dim] (heads of a group share them), v [tokens, heads * vdim], views with unit inner
     stride of one dtype.  Per key channel (default): z [tokens, heads * dim] (of that dtype or float32), a = sigmoid(z + bias)^(1 / tau), c = 1.
     ``per_head``: z [tokens, heads], dt = softplus(z + bias), a = exp(-exp(a_log) dt) for all of the head's channels, c = dt.
+    ``floor`` (float32 [heads * dim]): z [tokens, heads * dim], a = floor + (1 - floor) sigmoid(z + bias) and 1 - a takes the place
+    of c k (``k`` is None).  ``q_silu``: q passes silu first.
     ``given`` = (a, c), float32 [tokens, heads] each: the decay and the factor on k per head, ready-made (z and bias are None).
     ``ones_col``: the value rows are narrower than the state, v [tokens, heads * v_cols] with v_cols < vdim, and the state's
     column v_cols is fed the constant 1 as a value (the columns after it 0): that column of the state is then the sum of the
@@ -1489,7 +1570,10 @@ def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: 
     if ones_col and not v_cols < vdim:
         raise KernelError("gated_scan: the column of ones needs a state wider than the value rows")
     q_ptr, q_stride = _scan_view(q, "q", groups * dim, dtype)
-    k_ptr, k_stride = _scan_view(k, "k", groups * dim, dtype)
+    if (k is None) != (floor is not None) or (floor is not None and (floor.dtype != torch.float32 or floor.numel() != heads * dim
+                                                                     or groups != heads or per_head or given is not None)):
+        raise KernelError("gated_scan: a forget gate with a floor has no keys, float32 floors [heads * dim] and query vectors per head")
+    k_ptr, k_stride = (None, 0) if k is None else _scan_view(k, "k", groups * dim, dtype)
     v_ptr, v_stride = _scan_view(v, "v", heads * v_cols, dtype)
     if given is not None:
         per_head = True
@@ -1523,13 +1607,52 @@ def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: 
     if given is not None:
         da, dc = given
     _run("sprout_gated_scan", q_ptr, q_stride, k_ptr, k_stride, v_ptr, v_stride, z_ptr, z_stride, 1 if z_f32 else 0,
-         _dtype_code(dtype), _ptr(bias, "bias", torch.float32, True), _ptr(a_log, "a_log", torch.float32, True), _ptr(skip, "skip", torch.float32, True),
-         1.0 / float(tau), float(q_scale), 2 if given is not None else 1 if per_head else 0, state.slots.numel(), heads, groups, dim, vdim,
+         _dtype_code(dtype), _ptr(bias, "bias", torch.float32, True), _ptr(a_log if floor is None else floor, "a_log", torch.float32, True), _ptr(skip, "skip", torch.float32, True),
+         1.0 / float(tau), float(q_scale), 2 if given is not None else 3 if floor is not None else 1 if per_head else 0, state.slots.numel(), heads, groups, dim, vdim,
          _ptr(ctx.q_start, "q_start", torch.int32), _ptr(state.slots, "state_slots", torch.int32),
          _ptr(buffer, "state", torch.float32), buffer.shape[0], _ptr(out, "out", torch.float32),
          _ptr(status, "status", torch.int32), tokens, SCAN_CHUNK, max_chunks, _ptr(da, "decays", torch.float32, True),
          _ptr(dc, "steps", torch.float32, True), _ptr(sums, "sums", torch.float32, True), _ptr(prods, "products", torch.float32, True),
-         v_cols, 1 if ones_col else 0, _stream())
+         v_cols, 1 if ones_col else 0, 1 if q_silu else 0, _stream())
+
+
+DELTA_CHUNK = 64            # tokens of a chunk of the delta rule
+DELTA_CHUNKED_FROM = 24     # a step whose longest portion has at least this many tokens runs the chunked form
+
+
+def delta_rule(q, k, v, b, a, a_log, dt_bias, ctx, state, out, heads: int, groups: int, dim: int, vdim: int, status,
+               q_scale: float = 1.0, unit_eps: float = 1e-6):
+    """The gated delta rule over the step's tokens, from and into the requests' state slots: per head, with unit-length q
+    (times ``q_scale``) and k shared by the heads of a group, g = exp(-exp(a_log) softplus(a + dt_bias)) and beta = sigmoid(b):
+    S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q.  q, k [tokens, groups * dim] and v [tokens, heads * vdim] are views
+    of one row stride, b and a [tokens, heads] likewise, all of one dtype; the state float32 [slots, heads, dim, vdim], out
+    float32 [tokens, heads * vdim].  A step whose longest portion has ``DELTA_CHUNKED_FROM`` tokens or more works in chunks of
+    ``DELTA_CHUNK`` tokens (``SPROUT_DELTA_RULE=walk`` keeps the walk from token to token)."""
+    tokens, dtype = v.shape[0], v.dtype
+    for name, t, width in (("q", q, groups * dim), ("k", k, groups * dim), ("v", v, heads * vdim), ("b", b, heads), ("a", a, heads)):
+        if t.dim() != 2 or t.stride(1) != 1 or tuple(t.shape) != (tokens, width) or t.dtype != dtype:
+            raise KernelError(f"delta_rule: {name} must be a [tokens, {width}] view with unit inner stride of {dtype}")
+    if not (q.stride(0) == k.stride(0) == v.stride(0)) or a.stride(0) != b.stride(0):
+        raise KernelError("delta_rule: q, k and v share one row stride, the two gates' inputs another")
+    buffer = state.buffer
+    if buffer.dtype != torch.float32 or not buffer.is_contiguous() or tuple(buffer.shape[1:]) != (heads, dim, vdim):
+        raise KernelError("delta_rule: state must be contiguous float32 [slots, heads, dim, vdim]")
+    if not out.is_contiguous() or out.dtype != torch.float32 or tuple(out.shape) != (tokens, heads * vdim) \
+            or a_log.numel() != heads or dt_bias.numel() != heads or dim > 256:
+        raise KernelError("delta_rule: out must be contiguous float32 [tokens, heads * vdim], one decay rate and bias per head, dim at most 256")
+    global LAUNCHES
+    requests, max_chunks, scratch = state.slots.numel(), 0, None
+    if getattr(ctx, "max_q_len", 1) >= DELTA_CHUNKED_FROM and os.environ.get("SPROUT_DELTA_RULE", "chunks") != "walk":
+        max_chunks = tokens // DELTA_CHUNK + requests
+        floats = (_lib or load_library()).sprout_delta_scratch_floats(max_chunks, heads, dim, vdim)
+        scratch = torch.empty(floats, dtype=torch.float32, device=v.device)
+        LAUNCHES += 2                                          # three kernels behind the call
+    _run("sprout_delta_rule", q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), b.data_ptr(), a.data_ptr(), a.stride(0),
+         _dtype_code(dtype), _ptr(a_log, "a_log", torch.float32), _ptr(dt_bias, "dt_bias", torch.float32), requests, heads, groups,
+         dim, vdim, float(q_scale), float(unit_eps), _ptr(ctx.q_start, "q_start", torch.int32),
+         _ptr(state.slots, "state_slots", torch.int32), _ptr(buffer, "state", torch.float32), buffer.shape[0],
+         _ptr(out, "out", torch.float32), max_chunks, _ptr(scratch, "scratch", torch.float32, True),
+         _ptr(status, "status", torch.int32), _stream())
 
 
 def causal_conv(rows, weight, bias, out, ctx, state, status, silu: bool = True):
@@ -1556,13 +1679,15 @@ def gated_group_norm(o, gate, weight, out, eps: float, groups: int = 1, gate_fir
     """Rows of ``o`` (float32 [rows, width]) in ``groups`` equal parts, each divided by its root mean square (eps inside
     the root), times ``weight`` (float32; it repeats every weight.numel() elements: a weight per head, or one for the whole
     row), times act(gate), act = silu or sigmoid; with ``gate_first`` the gate is applied before the norm.  ``gate`` is a
-    [rows, width] view with unit inner stride of out's dtype."""
-    _rows_contiguous(gate, "gate")
+    [rows, width] view with unit inner stride of out's dtype, or None (no gate)."""
+    if gate is not None:
+        _rows_contiguous(gate, "gate")
     rows, width = o.shape
     if not o.is_contiguous() or o.dtype != torch.float32 or not out.is_contiguous() or out.shape != o.shape \
-            or gate.shape != o.shape or gate.dtype != out.dtype or width % weight.numel() or width % groups:
+            or (gate is not None and (gate.shape != o.shape or gate.dtype != out.dtype)) or (gate is None and gate_first) \
+            or width % weight.numel() or width % groups:
         raise KernelError("gated_group_norm: shapes or dtypes do not fit")
-    _run("sprout_gated_group_norm", _ptr(o, "o", torch.float32), _ptr(gate, "gate"), gate.stride(0),
+    _run("sprout_gated_group_norm", _ptr(o, "o", torch.float32), _ptr(gate, "gate", allow_none=True), 0 if gate is None else gate.stride(0),
          _ptr(weight, "weight", torch.float32), weight.numel(), _ptr(out, "out"), _dtype_code(out.dtype), rows, width,
          int(groups), float(eps), 1 if gate_first else 0, 1 if silu else 0, _stream())
 
@@ -1679,6 +1804,15 @@ def rms_add(y, weight, x, eps: float):
         raise KernelError("rms_add: contiguous float32 rows of one shape and a weight per column")
     _run("sprout_rms_add", _ptr(y, "y", torch.float32), _ptr(weight, "weight", torch.float32), _ptr(x, "x", torch.float32),
          x.shape[0], x.shape[1], float(eps), _stream())
+
+
+def rms_pair_add(y1, y2, w1, w2, x, eps: float, factor: float = 1.0):
+    """x += factor * (y1 / rms(y1) * w1 + y2 / rms(y2) * w2), row by row (eps inside the roots); float32."""
+    if any(t.dtype != torch.float32 or not t.is_contiguous() or t.shape != x.shape for t in (y1, y2, x)) \
+            or any(w.dtype != torch.float32 or w.numel() != x.shape[1] for w in (w1, w2)):
+        raise KernelError("rms_pair_add: contiguous float32 rows of one shape and a weight per column")
+    _run("sprout_rms_pair_add", _ptr(y1, "y1"), _ptr(y2, "y2"), _ptr(w1, "w1"), _ptr(w2, "w2"), _ptr(x, "x"), x.shape[0], x.shape[1],
+         float(eps), float(factor), _stream())
 
 
 def add_rows(x, vec, other=None):

@@ -93,11 +93,13 @@ class DecoderModel:
 
     def state_specs(self):
         """One StateSpec (or a tuple of them, or None) per state entry: entry i < len(layers) is layer i's own; a layer
-        call that names a further entry (a layer that runs several times, each run with a state of its own) adds it."""
+        call that names a further entry (a layer that runs several times, each run with a state of its own) adds it.  One more
+        entry, the last, is the embedding's."""
         specs = [block.mixer.state_spec() for block in self.blocks]
         further = {call.state: call.layer for call in self.spec.order if call.state is not None and call.state >= len(self.blocks)}
         for entry in range(len(self.blocks), max(further, default=-1) + 1):
             specs.append(specs[further[entry]] if entry in further else None)
+        specs.append(self.embedding.state_spec())               # the last entry is the embedding's own
         return specs
 
     def decode_plan(self, requests: int, max_keys: int, planned_context: int, page_tokens: int):
@@ -115,7 +117,7 @@ class DecoderModel:
         """Run the step's tokens through the layers in run order; float32 logits
         [len(ctx.logits_rows), vocab], or None when no logits are wanted.  ``storage`` is the device side of the cache
         (``cache.storage.CacheStorage``)."""
-        x = self.embedding.forward(ctx.token_ids)
+        x = self.embedding.forward(ctx.token_ids, ctx, storage.state_view(-1, ctx))
         carry = self.stream.begin(x, len(self.spec.order)) if self.stream else None
         # a block that ends in a norm may hand that norm to the stream part, which then also fills what the next block reads
         fuses = self.stream is not None and hasattr(self.stream, "norm_after")

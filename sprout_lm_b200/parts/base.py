@@ -22,7 +22,8 @@ Categories and what each must provide:
 * ``feed_forward``:  ``forward(h, x, ctx)``: adds its output to ``x`` in place.
 * ``block``:         arranges a layer's norms, mixer and feed-forward:
                      ``forward(x, ctx, cache, state)``.
-* ``embedding``:     ``forward(token_ids) -> x`` (float32 [tokens, hidden]).
+* ``embedding``:     ``forward(token_ids, ctx, state) -> x`` (float32 [tokens, hidden]); ``state_spec()`` as a mixer's (a
+                     row that also depends on the tokens before).
 * ``head``:          ``forward(h) -> logits`` (float32 [rows, vocab]).
 * ``stream``:        what goes from one layer call to the next when that is more than the layer's
                      result: ``begin(x, calls) -> carry`` after the embedding, ``after(carry, n, x)``

@@ -1,9 +1,18 @@
 """Arrangements of a layer's parts.  ``pre_norm``: x += mixer(norm_0(x)); x += ffn(norm_1(x))
-(src/qwen.ts:164-200); a layer without a feed-forward (``feed_forward.kind == "none"``) is the first half alone."""
+(src/qwen.ts:164-200); a layer without a feed-forward (``feed_forward.kind == "none"``) is the first half alone.
+``options["branch_scale"]`` multiplies what both sublayers add: the parts take it as their ``out_scale`` and fold it into
+a step they have anyway."""
 from __future__ import annotations
 
-from ..config.specs import LayerSpec
+from ..config.specs import LayerSpec, PartSpec
 from .base import Part, build_part, register_part
+
+
+def scaled(spec: PartSpec, factor: float) -> PartSpec:
+    """The part with its output multiplied by ``factor`` (its ``out_scale`` parameter)."""
+    if factor == 1.0:
+        return spec
+    return PartSpec(spec.kind, {**spec.params, "out_scale": factor * spec.params.get("out_scale", 1.0)})
 
 
 @register_part("block", "pre_norm")
@@ -13,8 +22,9 @@ class PreNormBlock(Part):
         if len(layer.norms) != (2 if self.has_ffn else 1):
             raise ValueError("a pre_norm block has one norm per sublayer")
         self.norms = [build_part("norm", spec, prefix) for spec in layer.norms]
-        self.mixer = build_part("mixer", layer.mixer, prefix)
-        self.feed_forward = build_part("feed_forward", layer.feed_forward, prefix) if self.has_ffn else None
+        branch = float(layer.options.get("branch_scale", 1.0))
+        self.mixer = build_part("mixer", scaled(layer.mixer, branch), prefix)
+        self.feed_forward = build_part("feed_forward", scaled(layer.feed_forward, branch), prefix) if self.has_ffn else None
 
     def parts(self):
         return [*self.norms, self.mixer, *([self.feed_forward] if self.has_ffn else [])]

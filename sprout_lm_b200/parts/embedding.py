@@ -6,7 +6,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
-from .base import Part, TensorDecl, WeightSource, register_part
+from .base import Part, StateSpec, TensorDecl, WeightSource, register_part
 from .linear import Linear
 
 
@@ -26,9 +26,45 @@ class TokenEmbedding(Part):
         self.table = source.matrix(self.tensor_name)
         self.runtime = source.runtime
 
-    def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
+    def state_spec(self):
+        return None
+
+    def forward(self, token_ids: torch.Tensor, ctx=None, state=None) -> torch.Tensor:
         x = torch.empty((token_ids.numel(), self.hidden_size), dtype=torch.float32, device=token_ids.device)
         kernels.embed(self.table, token_ids, x, self.runtime.status, scale=self.scale)
+        return x
+
+
+@register_part("embedding", "token_pair_embedding")
+class TokenPairEmbedding(TokenEmbedding):
+    """The token's row times ``scale`` plus a row of a second table that the last two tokens choose:
+    (previous * mul_prev + token * mul_cur) mod ``buckets``; a sequence's first token takes the table's last row (number
+    ``buckets``).  A request's last token is its state: int32 [1] in its slot."""
+
+    def __init__(self, prefix: str, vocab_size: int, hidden_size: int, buckets: int, mul_prev: int, mul_cur: int,
+                 pair_name: str = "bigram", **base):
+        super().__init__(prefix, vocab_size, hidden_size, **base)
+        if buckets <= 0:
+            raise ValueError("token_pair_embedding: the table of pairs needs at least one row beside the first token's")
+        self.buckets, self.mul_prev, self.mul_cur = int(buckets), int(mul_prev), int(mul_cur)
+        self.pair_name = prefix + pair_name
+        self.pairs = None
+
+    def tensor_decls(self):
+        return super().tensor_decls() + [TensorDecl(self.pair_name, (self.buckets + 1, self.hidden_size))]
+
+    def load(self, source: WeightSource):
+        super().load(source)
+        self.pairs = source.matrix(self.pair_name)
+
+    def state_spec(self):
+        return StateSpec(shape=(1,), dtype=torch.int32)
+
+    def forward(self, token_ids: torch.Tensor, ctx=None, state=None) -> torch.Tensor:
+        if ctx is None or state is None:
+            raise RuntimeError("token_pair_embedding: the previous tokens live in the requests' state slots")
+        x = torch.empty((token_ids.numel(), self.hidden_size), dtype=torch.float32, device=token_ids.device)
+        kernels.embed_pairs(self.table, self.pairs, ctx, state, x, self.scale, self.mul_prev, self.mul_cur, self.runtime.status)
         return x
 
 

@@ -1,6 +1,6 @@
 """Recurrent mixers whose decay is made from the input: a float32 state per request and head, no keys or values per token.
 
-Both run S_t = diag(a_t) S_(t-1) + (c_t k_t) v_t^T, o_t = S_t^T q_t per head on the same scan kernel
+All run S_t = diag(a_t) S_(t-1) + (c_t k_t) v_t^T, o_t = S_t^T q_t per head on the same scan kernel
 (``csrc/gated_recurrence.cu``); the state [heads, dim, value_dim] starts at zero, is float32 and lives in the request's
 state slot.  Everything that enters the recurrence beside the projections (decays and their logarithms, softplus,
 exponentials, step sizes, norms) is float32 in both compute dtypes.
@@ -16,6 +16,11 @@ start of the sequence) and silu; dt = softplus(dt + dt_bias); per head (head h r
 a = exp(-exp(A_log_h) dt) for all of the head's rows, c = dt, k = B, q = C, v = x, and o gets D_h x added.  The heads side
 by side are multiplied by silu(z), then divided in ``norm_groups`` equal parts by each part's root mean square and
 multiplied by a weight [inner], then projected by W_o.  The convolution's last taps - 1 inputs are a second state tensor.
+
+``forget_write_attention`` (the HGRN2 recurrence): q = silu(W_q h), v = W_v h; a forget gate per head and channel with a lower bound,
+f = lower + (1 - lower) sigmoid(W_f h + b_f) (heads x dim); a = f, and c k = 1 - f: what is not kept is written, there is no
+key.  Each head's o is divided by its root mean square over value_dim and multiplied by a weight [value_dim] that the heads
+share; the heads side by side are projected by W_o.
 
 ``out_scale`` multiplies the mixer's output (it is folded into the norm's weight), so that a block that runs several
 mixers side by side can weigh them without a kernel of its own.
@@ -154,3 +159,52 @@ class SelectiveStateSpace(Part):
         kernels.gated_group_norm(y, rows[:, :inner], self.gain, gated, self.eps, groups=self.norm_groups, gate_first=True,
                                  silu=True)
         self.out.forward(gated, residual=x)
+
+
+@register_part("mixer", "forget_write_attention")
+class ForgetWriteAttention(Part):
+    DEFAULT_NAMES = {"q": "q", "f": "f", "f_bias": "f.b", "lower": "lower", "v": "v", "norm": "norm", "o": "o"}
+
+    def __init__(self, prefix: str, hidden_size: int, heads: int, dim: int, value_dim: int, eps: float, out_scale: float = 1.0,
+                 names: dict | None = None):
+        if hidden_size <= 0 or heads <= 0 or dim <= 0 or value_dim <= 0 or eps <= 0:
+            raise ValueError("forget_write_attention: sizes and eps must be positive")
+        self.hidden_size, self.heads, self.dim, self.value_dim = hidden_size, heads, dim, value_dim
+        self.eps, self.out_scale = float(eps), float(out_scale)
+        self.names = {key: prefix + value for key, value in {**self.DEFAULT_NAMES, **(names or {})}.items()}
+        self.runtime = None
+
+    def cache_spec(self):
+        return None
+
+    def state_spec(self):
+        return StateSpec(shape=(self.heads, self.dim, self.value_dim), dtype=torch.float32)
+
+    def tensor_decls(self):
+        n, qk, vw = self.names, self.heads * self.dim, self.heads * self.value_dim
+        return [TensorDecl(n["q"], (qk, self.hidden_size)), TensorDecl(n["f"], (qk, self.hidden_size)),
+                TensorDecl(n["f_bias"], (qk,), "bias"), TensorDecl(n["lower"], (qk,), "bias"),
+                TensorDecl(n["v"], (vw, self.hidden_size)), TensorDecl(n["norm"], (self.value_dim,), "gain"),
+                TensorDecl(n["o"], (self.hidden_size, vw))]
+
+    def load(self, source: WeightSource):
+        n, status = self.names, source.runtime.status
+        self.runtime = source.runtime
+        fused = torch.cat([source.raw(n[key]) for key in ("q", "f", "v")], dim=0)
+        self.proj = Linear(source.to_device_matrix(fused), None, status, any_inner_size=True)
+        self.bias, self.lower = source.vector(n["f_bias"]), source.vector(n["lower"])
+        self.gain = (source.vector(n["norm"]) * self.out_scale).contiguous()
+        self.out = Linear(source.matrix(n["o"]), None, status, any_inner_size=True)
+
+    def forward(self, h, x, ctx, cache, state: StateView):
+        """x (float32) += out_scale * W_o (rmsnorm_per_head(o) * w); the requests' states advance."""
+        if state is None:
+            raise RuntimeError("forget_write_attention: the layer needs a state slot per request")
+        rows = self.proj.forward(h)
+        qk, vw = self.heads * self.dim, self.heads * self.value_dim
+        o = torch.empty((rows.shape[0], vw), dtype=torch.float32, device=rows.device)
+        kernels.gated_scan(rows[:, :qk], None, rows[:, 2 * qk:2 * qk + vw], rows[:, qk:2 * qk], self.bias, ctx, state, o, self.heads,
+                           self.heads, self.dim, self.value_dim, self.runtime.status, floor=self.lower, q_silu=True)
+        normed = torch.empty((rows.shape[0], vw), dtype=rows.dtype, device=rows.device)
+        kernels.gated_group_norm(o, None, self.gain, normed, self.eps, groups=self.heads)
+        self.out.forward(normed, residual=x)

@@ -255,7 +255,9 @@ class RoutedExperts(Part):
     times ``scale``; ``groups`` = (count, keep): the experts form ``count`` equal groups of neighbours, a group's score is
     its largest score, and only experts of the ``keep`` best groups can be taken; ``shared_gate``: the shared expert's
     output is multiplied by sigmoid(w_sg . h), one number per token, its row ``shared.sg`` [1, hidden] multiplied in the
-    router's 32-bit product.
+    router's 32-bit product; ``expert_kind`` = "silu_glu": experts are W_down (silu(W_gate h) * W_up h); ``scores`` = "sigmoid":
+    s = sigmoid(z), each output for itself; ``weight_on`` = "input": an expert reads its weight times h and the outputs are
+    added as they are; ``out_scale`` multiplies what is added to x (without a shared expert).
 
     Tensors: ``router`` [experts + identity, hidden], ``correction`` [experts + identity], ``e<i>.gate|up|down``,
     ``shared.gate|up|down`` (no ``gate`` matrices for plain experts), ``shared.sg``."""
@@ -263,13 +265,20 @@ class RoutedExperts(Part):
     def __init__(self, prefix: str, hidden_size: int, experts: int, identity: int, top: int, scale: float, expert_ff: int,
                  expert_limit: float = 0.0, alpha: float = 1.702, shared_ff: int | None = None, shared_limit: float | None = None,
                  names: dict | None = None, expert_kind: str = "clamped_glu", correction: bool = True, renormalize: bool = True,
-                 groups=None, shared_gate: bool = False):
+                 groups=None, shared_gate: bool = False, scores: str = "softmax", weight_on: str = "output", out_scale: float = 1.0):
         if hidden_size <= 0 or experts < 0 or identity < 0 or experts + identity <= 0 or not 0 < top <= experts + identity:
             raise ValueError("routed_experts: bad sizes")
-        if expert_kind not in ("clamped_glu", "plain"):
-            raise ValueError("routed_experts: experts are 'clamped_glu' or 'plain'")
+        if expert_kind not in kernels.EXPERT_UNITS:
+            raise ValueError(f"routed_experts: experts are one of {', '.join(kernels.EXPERT_UNITS)}")
+        if scores not in ("softmax", "sigmoid") or weight_on not in ("output", "input"):
+            raise ValueError("routed_experts: scores are 'softmax' or 'sigmoid', the weight is on the 'output' or the 'input'")
+        if shared_ff is not None and (expert_kind == "silu_glu" or out_scale != 1.0):
+            raise ValueError("routed_experts: a shared expert is clamped or plain, and not scaled")
+        if identity and weight_on == "input":
+            raise ValueError("routed_experts: identity experts take their weight on the output")
+        self.expert_kind, self.sigmoid, self.weight_on_input, self.out_scale = expert_kind, scores == "sigmoid", weight_on == "input", float(out_scale)
         self.plain = expert_kind == "plain"
-        if experts and (expert_ff <= 0 or (not self.plain and expert_limit <= 0)):
+        if experts and (expert_ff <= 0 or (expert_kind == "clamped_glu" and expert_limit <= 0)):
             raise ValueError("routed_experts: experts need a positive size and limit")
         if shared_ff is not None and (shared_ff <= 0 or (not self.plain and (shared_limit is None or shared_limit <= 0))):
             raise ValueError("routed_experts: a shared expert needs a positive size and limit")
@@ -281,8 +290,8 @@ class RoutedExperts(Part):
         if shared_gate and shared_ff is None:
             raise ValueError("routed_experts: a gate without a shared expert")
         self.has_correction, self.renormalize, self.groups, self.shared_gate = bool(correction), bool(renormalize), groups, bool(shared_gate)
-        if self.plain:
-            expert_limit = 0.0           # what tells the experts' kernels that there is no gate
+        if expert_kind != "clamped_glu":
+            expert_limit = 0.0
         self.hidden_size, self.experts, self.identity, self.top = hidden_size, experts, identity, top
         self.scale, self.expert_ff, self.expert_limit, self.alpha = float(scale), expert_ff, float(expert_limit), float(alpha)
         self.shared_ff, self.shared_limit = shared_ff, shared_limit
@@ -344,8 +353,10 @@ class RoutedExperts(Part):
         ids = torch.empty((tokens, self.top), dtype=torch.int32, device=device)
         weights = torch.empty((tokens, self.top), dtype=torch.float32, device=device)
         gate_logits = torch.empty((tokens, 1), dtype=torch.float32, device=device) if self.shared_gate else None
-        kernels.moe_route(h, self.router, self.correction, ids, weights, self.counts, self.experts, self.top, self.scale,
-                          groups=self.groups, renormalize=self.renormalize, extra_out=gate_logits)
+        # a factor on the output goes onto the weights, unless they go into the experts
+        scale = self.scale if self.weight_on_input else self.scale * self.out_scale
+        kernels.moe_route(h, self.router, self.correction, ids, weights, self.counts, self.experts, self.top, scale,
+                          groups=self.groups, renormalize=self.renormalize, extra_out=gate_logits, sigmoid=self.sigmoid)
         place_of = torch.empty(entries, dtype=torch.int32, device=device)
         rows = None
         if self.experts:
@@ -354,7 +365,7 @@ class RoutedExperts(Part):
             act = torch.empty((entries, self.expert_ff), dtype=h.dtype, device=device)
             rows = torch.empty((entries, self.hidden_size), dtype=torch.float32, device=device)
             kernels.moe_experts(h, order, self.offsets, self.w_gate_up, self.w_down, act, rows, self.experts, self.top,
-                                self.expert_limit, self.alpha)
+                                self.expert_limit, self.alpha, unit=self.expert_kind, row_weights=weights if self.weight_on_input else None)
         else:
             place_of.fill_(-1)
         if self.shared is not None and self.shared_gate and self.plain:
@@ -365,4 +376,4 @@ class RoutedExperts(Part):
             kernels.gated_rows_add(x, y, gate_logits)
         elif self.shared is not None:
             self.shared.forward(h, x)
-        kernels.moe_combine(x, h, ids, weights, place_of, rows, self.top)
+        kernels.moe_combine(x, h, ids, None if self.weight_on_input else weights, place_of, rows, self.top, factor=self.out_scale)

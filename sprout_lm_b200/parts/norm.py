@@ -2,7 +2,7 @@
 
 ``offset`` is added to the stored weight to give the gain: 0 for a weight stored around one, 1 for a
 weight stored around zero (gain = 1 + w).  ``suffix`` is what follows the part's name in the
-checkpoint's tensor name."""
+checkpoint's tensor name.  ``one_number``: the stored weight is a single number that serves every element."""
 from __future__ import annotations
 
 import torch
@@ -15,19 +15,23 @@ from .base import Part, TensorDecl, WeightSource, register_part
 class RMSNorm(Part):
     fused_kind = "rmsnorm"       # a consumer that has this norm's arithmetic in its own kernel may take gain and eps
 
-    def __init__(self, prefix: str, size: int, eps: float, name: str = "norm", offset: float = 0.0, suffix: str = ".weight"):
+    def __init__(self, prefix: str, size: int, eps: float, name: str = "norm", offset: float = 0.0, suffix: str = ".weight",
+                 one_number: bool = False):
         if eps <= 0:
             raise ValueError("rmsnorm: eps must be positive")
         self.size, self.eps, self.offset = int(size), float(eps), float(offset)
+        self.one_number = bool(one_number)
         self.tensor_name = f"{prefix}{name}{suffix}"
         self.gain = None
         self.out_dtype = None
 
     def tensor_decls(self):
-        return [TensorDecl(self.tensor_name, (self.size,), "gain" if self.offset == 0.0 else "bias")]
+        return [TensorDecl(self.tensor_name, () if self.one_number else (self.size,), "gain" if self.offset == 0.0 else "bias")]
 
     def load(self, source: WeightSource):
         self.gain = source.vector(self.tensor_name)
+        if self.one_number:
+            self.gain = self.gain.reshape(1).expand(self.size).contiguous()      # the kernels multiply by a vector
         if self.offset:
             self.gain = (self.gain + self.offset).contiguous()
         self.out_dtype = source.runtime.dtype

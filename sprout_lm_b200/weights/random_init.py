@@ -29,7 +29,8 @@ def _generator(seed: int, name: str) -> np.random.Generator:
 
 
 def random_tensor(seed: int, name: str, shape, init: str) -> torch.Tensor:
-    values = _generator(seed, name).standard_normal(size=shape, dtype=np.float32) * np.float32(STD)
+    values = np.asarray(_generator(seed, name).standard_normal(size=shape, dtype=np.float32), dtype=np.float32).reshape(shape) * np.float32(STD)
+    values = np.asarray(values, dtype=np.float32)               # a tensor without dimensions stays an array
     if init == "gain":
         values += np.float32(1.0)
     elif init == "pass_last":
