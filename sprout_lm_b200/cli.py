@@ -1,8 +1,8 @@
 """Command line in the manner of the reference's demo (src/demo.ts) and smoke script
 (scripts/smoke-cuda.ts).
 
-    python -m sprout_lm_b200 demo [--model DIR | --tiny A|B|T|L|V] [--seed S] [--json] [--pressure] [--dtype bfloat16|float32]
-    python -m sprout_lm_b200 generate (--model DIR | --tiny A|B|T|L|V) --prompt 1,2,3 [--max-new-tokens N]
+    python -m sprout_lm_b200 demo [--model DIR | --tiny A|B|T|L|V|Z] [--seed S] [--json] [--pressure] [--dtype bfloat16|float32]
+    python -m sprout_lm_b200 generate (--model DIR | --tiny A|B|T|L|V|Z) --prompt 1,2,3 [--max-new-tokens N]
                                       [--temperature T] [--seed S] [--ignore-eos] [--json]
     python -m sprout_lm_b200 random-model --out DIR --config CONFIG.json [--seed S]
 
@@ -86,6 +86,24 @@ TINY_CONFIGS["V"] = {
                         "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}},
                {"type": "attention", "mixer": {"heads": 4, "kv_heads": 1, "dim": 32, "vdim": 64, "scale": 0.2, "softcap": 15.0},
                 "mlp": {"kind": "dense", "ff": 160}}]}
+
+
+# --tiny Z: a tiny random Zevedra model (windowed attention with turned values beside the gated delta rule; full attention with a
+# gate per element beside a recurrence whose forget gate writes; experts weighed on their input; the last two layers run twice;
+# a row of the last two tokens joins the embedding)
+TINY_CONFIGS["Z"] = {
+    "architecture": "Zevedra", "vocab": 384, "width": 128, "norm": {"eps": 1e-5}, "residual_mult": 0.8, "max_positions": 512,
+    "embedding": {"scale": 11.0, "bigram": {"buckets": 499, "mul_prev": 13, "mul_cur": 7}}, "loop": {"start": 1, "stop": 3, "times": 2},
+    "layers": [{"type": kind, "mixer": mixer, "mlp": {"kind": "moe", "expert": {"ff": 48}, "router": {"experts": 8, "top": 2}}}
+               for kind, mixer in (
+                   ("parallel", {"left": {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 64, "conv": 3, "mask": {"size": 20}, "scale": 0.2,
+                                          "rot": {"base": 10000.0, "dims": 16}}, "left_scale": 0.7,
+                                 "right": {"heads": 2, "kv_heads": 1, "dim": 32, "vdim": 32, "conv": 4}, "right_scale": 0.8}),
+                   ("parallel_2", {"left": {"heads": 2, "kv_heads": 2, "dim": 64, "vdim": 64, "scale": 0.125,
+                                            "rot": {"base": 10000.0, "dims": 64}}, "right": {"heads": 2, "dim": 32, "vdim": 48}}),
+                   ("parallel", {"left": {"heads": 4, "kv_heads": 1, "dim": 32, "vdim": 32, "conv": 2, "mask": {"size": 9}, "scale": 0.2,
+                                          "rot": {"base": 500.0, "dims": 32}}, "left_scale": 0.5,
+                                 "right": {"heads": 2, "kv_heads": 2, "dim": 16, "vdim": 64, "conv": 2}, "right_scale": 1.0}))]}
 
 
 def _table(rows: list[dict]) -> str:
@@ -236,7 +254,7 @@ def main(argv=None) -> int:
         p.add_argument("--tiny", choices=sorted(TINY) + sorted(TINY_CONFIGS), help="instead of --model: a tiny random model (A: 2 layers, "
                        "hidden 64, 4/2 heads of 16, tied head; B: 3 layers, hidden 96, 3/1 heads of 32, untied head; T: a Tulipel "
                        "model of 4 latent-attention layers, width 128; L: a Letanex model of 3 layers, width 128; V: a Vuripel model of "
-                       "3 layers of which two run twice, width 128), written with --seed")
+                       "3 layers of which two run twice, width 128; Z: a Zevedra model of 3 layers of which two run twice, width 128), written with --seed")
         p.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16")
         p.add_argument("--seed", type=int, default=0)
     rnd = sub.add_parser("random-model", help="write config.json and model.safetensors with random weights")

@@ -183,7 +183,7 @@ class ForgetWriteAttention(Part):
     def tensor_decls(self):
         n, qk, vw = self.names, self.heads * self.dim, self.heads * self.value_dim
         return [TensorDecl(n["q"], (qk, self.hidden_size)), TensorDecl(n["f"], (qk, self.hidden_size)),
-                TensorDecl(n["f_bias"], (qk,), "bias"), TensorDecl(n["lower"], (qk,), "bias"),
+                TensorDecl(n["f_bias"], (qk,), "bias"), TensorDecl(n["lower"], (qk,), "share"),
                 TensorDecl(n["v"], (vw, self.hidden_size)), TensorDecl(n["norm"], (self.value_dim,), "gain"),
                 TensorDecl(n["o"], (self.hidden_size, vw))]
 
