@@ -1462,6 +1462,228 @@ def timed_vuripel(args) -> dict:
     return result
 
 
+ZEVEDRA_SHAPES = {
+    "1b": dict(width=2048, heads=16, kv_heads=4, win_dim=64, win_vdim=128, window=1024, taps=4, dim=128, vdim=128, delta_heads=16,
+               delta_kv=8, delta_dim=128, delta_vdim=128, write_heads=16, write_dim=128, write_vdim=128, experts=32, top=4, expert_ff=1024,
+               buckets=65521, vocab=32768),
+    "0.3b": dict(width=1024, heads=8, kv_heads=2, win_dim=64, win_vdim=128, window=512, taps=4, dim=128, vdim=128, delta_heads=8,
+                 delta_kv=4, delta_dim=128, delta_vdim=128, write_heads=8, write_dim=128, write_vdim=128, experts=16, top=4, expert_ff=512,
+                 buckets=65521, vocab=32768),
+}
+
+
+def zevedra_folders(shape: str, layers: int):
+    """(Zevedra folder, Vuripel folder, Rarutar folder of equal size), random weights, written once.  Zevedra's layers in turn: a
+    window beside the gated delta rule, attention over everything beside the recurrence whose forget gate writes; routed experts
+    everywhere; all layers form one pass of a loop.  Vuripel (``--only vuripel``'s model: routed experts, attention, a matrix
+    memory) and Rarutar (pairs of mixers) beside it at the same width, heads, window, experts and vocabulary."""
+    from sprout_lm_b200 import parse_config, write_random_model
+    z = ZEVEDRA_SHAPES[shape]
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    first = {"left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["win_dim"], "vdim": z["win_vdim"], "scale": z["win_dim"] ** -0.5,
+                      "conv": z["taps"], "mask": {"size": z["window"]}, "rot": {"base": 500000.0, "dims": z["win_dim"]}},
+             "right": {"heads": z["delta_heads"], "kv_heads": z["delta_kv"], "dim": z["delta_dim"], "vdim": z["delta_vdim"], "conv": z["taps"]},
+             "left_scale": 0.5, "right_scale": 0.5}
+    second = {"left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+                       "rot": {"base": 500000.0, "dims": z["dim"]}},
+              "right": {"heads": z["write_heads"], "dim": z["write_dim"], "vdim": z["write_vdim"]}}
+    raw = {"architecture": "Zevedra", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.8,
+           "embedding": {"scale": 1.0, "bigram": {"buckets": z["buckets"], "mul_prev": 40961, "mul_cur": 257}},
+           "loop": {"start": 0, "stop": layers, "times": 1}, "max_positions": 16384,
+           "layers": [{"type": ("parallel", "parallel_2")[i % 2], "mixer": (first, second)[i % 2], "mlp": moe} for i in range(layers)]}
+    folder = Path(tempfile.gettempdir()) / f"sprout_lm_b200_bench_{os.getuid()}_zevedra_{shape}_L{layers}"
+    if not (folder / "complete").exists():
+        print(f"[bench] writing random weights to {folder}", file=sys.stderr, flush=True)
+        write_random_model(folder, parse_config(raw), seed=0)
+        (folder / "complete").write_text("ok")
+    return (folder, *vuripel_folders(shape, layers))
+
+
+def timed_zevedra_kernels(shape: str, tokens: int, batch: int, context: int, peak: dict) -> dict:
+    """Zevedra's kernels alone beside the like kernels of the closest models at equal sizes, for one prompt of ``tokens`` tokens
+    and for ``batch`` single tokens with ``context`` keys held.  Attention over a window with turned values beside Rarutar's
+    window, attention over everything with one added to the denominator and a gate per element beside Rarutar's with a sink and a
+    gate per head (executed FLOPs of the visible keys against the measured bf16 rate; bytes of the visible keys against the
+    measured copy rate).  The delta rule beside the scan with a decay per head, the forget gate that writes beside the scan with a
+    decay per channel (operations of the recurrence against the CUDA cores' nominal rate; bytes against the copy rate).  The
+    convolution of the projections, the append with norms and turned values, the pair of normed outputs, the experts, the router
+    and the embedding beside the plainer forms of each."""
+    import torch
+    from types import SimpleNamespace
+    from sprout_lm_b200 import kernels
+    z = ZEVEDRA_SHAPES[shape]
+    page, width = 16, z["width"]
+    g = torch.Generator(device="cuda").manual_seed(0)
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    out = {}
+
+    def rand(*shape_, scale=1.0, dtype=torch.bfloat16):
+        return (torch.randn(*shape_, device="cuda", generator=g) * scale).to(dtype)
+
+    def moved(name, us, mb, **more):
+        out[name] = {"us": round(us, 1), "mb": round(mb, 2), "gbs": round(mb / us * 1e3), "of_measured_copy": round(mb / us * 1e3 / peak["hbm_gbs"], 3),
+                     **more}
+    try:
+        top_mhz = float(subprocess.run(["nvidia-smi", "--query-gpu=clocks.max.sm", "--format=csv,noheader,nounits", "-i", "0"],
+                                       capture_output=True, text=True, timeout=20).stdout.split()[0])
+    except (OSError, ValueError, IndexError, subprocess.SubprocessError):
+        top_mhz = 1965.0
+    fp32_tflops = torch.cuda.get_device_properties(0).multi_processor_count * 128 * 2 * top_mhz / 1e6
+    out["fp32_cuda_core_tflops_nominal"] = round(fp32_tflops, 1)
+    heads, kv = z["heads"], z["kv_heads"]
+    turn = (torch.ones(16384, z["win_vdim"] // 2, device="cuda"), torch.zeros(16384, z["win_vdim"] // 2, device="cuda"))
+    key_turn = (torch.ones(16384, z["win_dim"] // 2, device="cuda"), torch.zeros(16384, z["win_dim"] // 2, device="cuda"))
+    for label, requests, new, held in (("prefill", 1, tokens, tokens), ("decode", batch, 1, context)):
+        n, repeats = requests * new, 3 if new > 1 else 10
+        pages = -(-held // page)
+        table = torch.full((requests, -(-pages // 64) * 64), -1, dtype=torch.int32, device="cuda")
+        table[:, :pages] = torch.randperm(requests * pages, device="cuda", generator=g).to(torch.int32).reshape(requests, pages)
+        ctx = SimpleNamespace(seq_of_token=torch.arange(requests, dtype=torch.int32, device="cuda").repeat_interleave(new),
+                              positions=(torch.arange(new, dtype=torch.int32, device="cuda") + (held - new)).repeat(requests),
+                              q_start=(torch.arange(requests + 1, dtype=torch.int32, device="cuda") * new), max_q_len=new, max_context=held,
+                              planned_context=0, token_ids=torch.randint(0, z["vocab"], (n,), dtype=torch.int32, device="cuda", generator=g))
+        # attention
+        window = ("window", z["window"])
+        for name, dim, vdim, mask, unit_sink, gate_width, value_turn in (
+                ("window_turned", z["win_dim"], z["win_vdim"], window, False, heads, turn), ("rarutar_window", z["win_dim"], z["win_vdim"], window, False, heads, None),
+                ("full_element_gate", z["dim"], z["vdim"], None, True, heads * z["vdim"], None), ("rarutar_sink_gate", z["dim"], z["vdim"], None, True, heads, None),
+                ("full_96_element_gate", 96, 96, None, True, heads * 96, None)):
+            k2, v2 = rand(requests * pages + 1, kv, page, dim), rand(requests * pages + 1, kv, page, vdim)
+            rows = rand(n, heads * dim + -(-gate_width // 8) * 8, scale=0.3)
+            o2 = torch.empty(n, heads * vdim, dtype=torch.bfloat16, device="cuda")
+            view = SimpleNamespace(k=k2, v=v2, block_table=table, page_tokens=page, write=False)
+            sink = torch.zeros(heads, device="cuda") if unit_sink else None
+            us = _median_us(lambda: kernels.multimap_attention(rows[:, :heads * dim], view, ctx, o2, heads, kv, 1, dim, vdim, dim ** -0.5, 0.0, 0.0, 1.0,
+                                                               status, mask=mask, sink=sink, gate=rows[:, heads * dim:heads * dim + gate_width],
+                                                               turn=value_turn, interleaved=True), repeats=repeats)
+            size = mask[1] if mask else held
+            if new > 1:
+                seen = sum(min(p + 1, size) for p in range(new))
+                tflops = 2.0 * heads * (dim + vdim) * seen / us / 1e6
+                out[f"{name}_{label}"] = {"us": round(us, 1), "tflops": round(tflops, 1), "of_measured_bf16": round(tflops / peak["bf16_tflops"], 3)}
+            else:
+                moved(f"{name}_{label}", us, batch * min(held, size) * kv * (dim + vdim) * 2 / 1e6)
+            del k2, v2, rows, o2
+        # norms, rotation, append: interleaved with turned values; over the whole projections; the plain form
+        dim, vdim = z["win_dim"], z["win_vdim"]
+        k2, v2 = rand(requests * pages + 1, kv, page, dim), rand(requests * pages + 1, kv, page, vdim)
+        rows = rand(n, heads * dim + kv * (dim + vdim))
+        qw, kw = torch.ones(heads * dim, device="cuda"), torch.ones(kv * dim, device="cuda")
+        mb = n * (heads * dim * 2 + kv * (dim + vdim) * 2) * 2 / 1e6
+        for name, options in (("append_turned", dict(unit_eps=1e-5, interleaved=True, value_turn=turn)), ("append_whole_norm", dict(q_weight=qw, k_weight=kw, weight_eps=1e-5)),
+                              ("append_rarutar", dict(unit_eps=1e-5)), ("append_vuripel", dict(q_weight=qw[:dim], k_weight=kw[:dim], weight_eps=1e-5))):
+            us = _median_us(lambda: kernels.rope_maps_append(rows, ctx.positions, ctx.seq_of_token, table, *key_turn, k2, v2, heads, kv, 1, dim, vdim, page,
+                                                             True, status, **options))
+            moved(f"{name}_{label}", us, mb)
+        # recurrences
+        slots = torch.arange(requests, dtype=torch.int32, device="cuda")
+        dh, dg, dd, dv = z["delta_heads"], z["delta_kv"], z["delta_dim"], z["delta_vdim"]
+        channels = 2 * dg * dd + dh * dv
+        proj = rand(n, channels + dh * dv + 2 * dh, scale=0.5)
+        conv = torch.empty(n, channels, dtype=torch.bfloat16, device="cuda")
+        taps = rand(channels, z["taps"], scale=0.3, dtype=torch.float32)
+        conv_state = SimpleNamespace(buffer=torch.zeros(requests, z["taps"] - 1, channels, device="cuda"), slots=slots)
+        for name, silu in (("conv_plain", False), ("conv_silu", True)):
+            us = _median_us(lambda: kernels.causal_conv(proj[:, :channels], taps, None, conv, ctx, conv_state, status, silu=silu))
+            moved(f"{name}_{label}", us, (n * channels * 4 + requests * channels * (z["taps"] - 1) * 8) / 1e6)
+        state = SimpleNamespace(buffer=torch.zeros(requests, dh, dd, dv, device="cuda"), slots=slots)
+        o = torch.empty(n, dh * dv, device="cuda")
+        a_log, bias = torch.full((dh,), -2.0, device="cuda"), torch.zeros(dh, device="cuda")
+        at, state_mb = channels + dh * dv, 2 * requests * dh * dd * dv * 4 / 1e6
+        us = _median_us(lambda: kernels.delta_rule(conv[:, :dg * dd], conv[:, dg * dd:2 * dg * dd], conv[:, 2 * dg * dd:], proj[:, at:at + dh],
+                                                   proj[:, at + dh:at + 2 * dh], a_log, bias, ctx, state, o, dh, dg, dd, dv, status,
+                                                   q_scale=dd ** -0.5), repeats=repeats)
+        moved(f"delta_rule_{label}", us, n * (channels * 2 + dh * 4 + dh * dv * 4) / 1e6 + state_mb,
+              of_nominal_fp32_cores=round(8.0 * n * dh * dd * dv / us / 1e6 / fp32_tflops, 3))      # two products with the state and a decayed update
+        us = _median_us(lambda: kernels.gated_scan(conv[:, :dg * dd], conv[:, dg * dd:2 * dg * dd], conv[:, 2 * dg * dd:], proj[:, at:at + dh], bias, ctx, state, o,
+                                                   dh, dg, dd, dv, status, per_head=True, a_log=a_log), repeats=repeats)
+        moved(f"head_decay_scan_{label}", us, n * (channels * 2 + dh * 2 + dh * dv * 4) / 1e6 + state_mb,
+              of_nominal_fp32_cores=round(6.0 * n * dh * dd * dv / us / 1e6 / fp32_tflops, 3))
+        wh, wd, wv = z["write_heads"], z["write_dim"], z["write_vdim"]
+        rows = rand(n, 3 * wh * wd + wh * wv, scale=0.5)
+        floor, zero = torch.full((wh * wd,), 0.5, device="cuda"), torch.zeros(wh * wd, device="cuda")
+        state = SimpleNamespace(buffer=torch.zeros(requests, wh, wd, wv, device="cuda"), slots=slots)
+        o = torch.empty(n, wh * wv, device="cuda")
+        state_mb = 2 * requests * wh * wd * wv * 4 / 1e6
+        for name, keys, options in (("forget_write_scan", None, dict(floor=floor, q_silu=True)), ("channel_decay_scan", rows[:, wh * wd:2 * wh * wd], dict(tau=16.0))):
+            us = _median_us(lambda: kernels.gated_scan(rows[:, :wh * wd], keys, rows[:, 3 * wh * wd:], rows[:, 2 * wh * wd:3 * wh * wd], zero, ctx, state, o, wh, wh,
+                                                       wd, wv, status, **options), repeats=repeats)
+            moved(f"{name}_{label}", us, n * ((3 if keys is not None else 2) * wh * wd * 2 + wh * wv * 6) / 1e6 + state_mb,
+                  of_nominal_fp32_cores=round(6.0 * n * wh * wd * wv / us / 1e6 / fp32_tflops, 3))
+        # rows: a norm per head with and without a gate, normed outputs, embedding
+        gain, gated = torch.ones(dv, device="cuda"), torch.empty(n, dh * dv, dtype=torch.bfloat16, device="cuda")
+        y = rand(n, dh * dv, dtype=torch.float32)
+        for name, gate in (("head_norm", None), ("gated_head_norm", proj[:, channels:channels + dh * dv])):
+            us = _median_us(lambda: kernels.gated_group_norm(y, gate, gain, gated, 1e-5, groups=dh))
+            moved(f"{name}_{label}", us, n * dh * dv * (6 if gate is None else 8) / 1e6)
+        x, y1, y2 = (rand(n, width, dtype=torch.float32) for _ in range(3))
+        ones = torch.ones(width, device="cuda")
+        moved(f"pair_norm_add_{label}", _median_us(lambda: kernels.rms_pair_add(y1, y2, ones, ones, x, 1e-5, 0.5)), n * width * 16 / 1e6)
+        moved(f"norm_add_{label}", _median_us(lambda: kernels.rms_add(y1, ones, x, 1e-5)), n * width * 12 / 1e6)
+        embed, pairs = rand(z["vocab"], width), rand(z["buckets"] + 1, width)
+        last = SimpleNamespace(buffer=torch.zeros(requests, 1, dtype=torch.int32, device="cuda"), slots=slots)
+        moved(f"embed_pairs_{label}", _median_us(lambda: kernels.embed_pairs(embed, pairs, ctx, last, x, 1.0, 40961, 257, status)), n * width * 8 / 1e6)
+        moved(f"embed_{label}", _median_us(lambda: kernels.embed(embed, ctx.token_ids, x, status)), n * width * 6 / 1e6)
+        del embed, pairs
+        # routed experts
+        experts, top, ff = z["experts"], z["top"], z["expert_ff"]
+        h, router = rand(n, width, scale=0.5), rand(experts, width, scale=0.05, dtype=torch.float32)
+        ids = torch.empty((n, top), dtype=torch.int32, device="cuda")
+        weights = torch.empty((n, top), dtype=torch.float32, device="cuda")
+        counts = torch.zeros(experts, dtype=torch.int32, device="cuda")
+        offsets = torch.zeros(experts + 1, dtype=torch.int32, device="cuda")
+        order, place_of = (torch.empty(n * top, dtype=torch.int32, device="cuda") for _ in range(2))
+        for name, sigmoid in (("softmax", False), ("sigmoid", True)):
+            def route():
+                kernels.moe_route(h, router, None, ids, weights, counts, experts, top, 1.0, renormalize=False, sigmoid=sigmoid)
+                kernels.moe_arrange(ids, counts, offsets, order, place_of, experts)
+            out[f"route_{name}_{label}"] = {"us": round(_median_us(route), 1)}
+        act = torch.empty((n * top, ff), dtype=torch.bfloat16, device="cuda")
+        rows_out = torch.empty((n * top, width), dtype=torch.float32, device="cuda")
+        w_up, w_down = rand(experts, 2 * ff, width, scale=0.02), rand(experts, width, ff, scale=0.02)
+        for name, options in (("silu_weighed", dict(unit="silu_glu", row_weights=weights)), ("clamped", dict(unit="clamped_glu"))):
+            us = _median_us(lambda: kernels.moe_experts(h, order, offsets, w_up, w_down, act, rows_out, experts, top, 7.0, 1.702, **options), repeats=repeats)
+            tflops = 6.0 * n * top * width * ff / us / 1e6
+            moved(f"experts_{name}_{label}", us, min(experts, n * top) * 3 * ff * width * 2 / 1e6, tflops=round(tflops, 1),
+                  of_measured_bf16=round(tflops / peak["bf16_tflops"], 3))
+        del w_up, w_down, act, rows_out
+    assert int(status.item()) == 0
+    return out
+
+
+def timed_zevedra(args) -> dict:
+    """``--only zevedra``: prefill and decode throughput of Zevedra at ``--shape 1b|0.3b`` (random weights, ``--layers`` layers,
+    4 if not given) beside Vuripel and Rarutar at equal size, through the same runner, and the kernels alone."""
+    import numpy as np
+    import torch
+    from sprout_lm_b200 import load_model
+    from sprout_lm_b200.engine.step import ModelRunner
+    shape = args.shape if args.shape in ZEVEDRA_SHAPES else "1b"
+    layers = args.layers or 4
+    peak = peaks()
+    folders = zevedra_folders(shape, layers)
+    prompt_len = args.prompt_len
+    result = {"impl": "ours", "only": "zevedra", "shape": shape, "layers": layers, "dtype": "bf16", "data": "synthetic",
+              "prefill_tokens": args.tokens, "decode_batch": args.batch, "decode_prompt_len": prompt_len, "steps": args.steps,
+              "peaks": {"bf16_tflops": peak["bf16_tflops"], "hbm_gbs": peak["hbm_gbs"], "source": peak.get("source", "measured")}}
+    for tag, folder in zip(("zevedra", "vuripel", "rarutar"), folders):
+        model = load_model(folder, dtype="bfloat16", device="cuda:0")
+        slots = max(64, args.batch)
+        pages = slots * (-(-(prompt_len + args.steps + args.warmup + 16) // 16)) + args.tokens // 16 + 16
+        runner = ModelRunner(model, num_pages=pages, page_tokens=16, max_requests=slots, prefix_caching=False)
+        rng = np.random.default_rng(0)
+        ms = timed_prefill(runner, args.tokens, rng)
+        decode = timed_decode(runner, args.batch, prompt_len, args.steps, args.warmup, rng)
+        result[tag] = {"weights_mb": round((folder / "model.safetensors").stat().st_size / 1e6, 1), "prefill_ms": round(ms, 3),
+                       "prefill_tokens_per_s": round(args.tokens / ms * 1000),
+                       "decode_ms_per_step": round(decode["ms_per_step"], 4), "decode_tokens_per_s": round(decode["tokens_per_s"]),
+                       "decode_launches_per_step": decode["launches_per_step"]}
+        del runner, model
+        torch.cuda.empty_cache()
+    result["kernels"] = timed_zevedra_kernels(shape, args.tokens, max(args.batch, 64), 2048, peak)
+    return result
+
+
 def run(args) -> dict:
     import numpy as np
     import torch
@@ -1477,6 +1699,8 @@ def run(args) -> dict:
         return timed_rarutar(args)
     if args.only == "vuripel":
         return timed_vuripel(args)
+    if args.only == "zevedra":
+        return timed_zevedra(args)
     if args.only == "attention":
         return timed_attention(args.tokens, args.shape)
     if args.only == "gemm":
@@ -1584,7 +1808,7 @@ def main() -> int:
     parser.add_argument("--portion", type=int, default=4096, help="with --only long-prompt: tokens of a step (--tokens: of the whole prompt)")
     parser.add_argument("--prompt-len", type=int, default=512, help="with --only decode: tokens of every request's prompt (the context grows to hold it)")
     parser.add_argument("--layers", type=int, default=0, help="fewer layers than the model has (named in config)")
-    parser.add_argument("--only", choices=["all", "decode", "prefill", "ablate", "attention", "decode-attention", "gemm", "serve", "long-prompt", "latent", "letanex", "rarutar", "vuripel"], default="all",
+    parser.add_argument("--only", choices=["all", "decode", "prefill", "ablate", "attention", "decode-attention", "gemm", "serve", "long-prompt", "latent", "letanex", "rarutar", "vuripel", "zevedra"], default="all",
                         help="measure one part only (for profiling captures); the JSON line then holds that part")
     parser.add_argument("--shape", choices=sorted(set(SHAPES) | set(LATENT_SHAPES) | set(LETANEX_SHAPES) | set(RARUTAR_SHAPES)), default="0.5b", help="with --only: the model's sizes")
     parser.add_argument("--requests", type=int, default=64, help="with --only serve: requests of the workload")

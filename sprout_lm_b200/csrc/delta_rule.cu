@@ -167,7 +167,7 @@ delta_walk_kernel(const DeltaParams<T> p, int slices_log2) {
 }
 
 // ------------------------------------------------------------------------------------------ chunks
-constexpr int DELTA_THREADS = 256, CARRY_COLS = 16, OUT_COLS = 64;
+constexpr int DELTA_THREADS = 256, CARRY_COLS = 16, CARRY_STRIDE = CARRY_COLS + 4, OUT_COLS = 64;   // rows of 20 floats: no two of 8 lanes' rows share a bank
 constexpr int PREP_A_STRIDE = DELTA_CHUNK + 4;
 
 // The chunks of all requests are numbered in the requests' order, ceil(tokens / 64) each.
@@ -194,14 +194,14 @@ __device__ __forceinline__ float dot4(const float4& a, const float4& b, float x)
 }
 
 template <typename T>
-__global__ void __launch_bounds__(DELTA_THREADS)
+__global__ void __launch_bounds__(DELTA_THREADS, 2)
 delta_prepare_kernel(const DeltaParams<T> p) {
   extern __shared__ float4 prep_smem[];
   const int dim = p.dim, dp = p.dim_pad, ds = dp + 4;
   float* kn = reinterpret_cast<float*>(prep_smem);        // [64][ds], unit keys
   float* qn = kn + DELTA_CHUNK * ds;                      // [64][ds], unit queries times q_scale
   float* at = qn + DELTA_CHUNK * ds;                      // [64][PREP_A_STRIDE]: at[j][i] = A_ij, zero for i <= j
-  __shared__ float s_beta[DELTA_CHUNK], s_g[DELTA_CHUNK];
+  __shared__ float s_beta[DELTA_CHUNK], s_g[DELTA_CHUNK], s_up[DELTA_CHUNK], s_down[DELTA_CHUNK];    // e^(G_i), e^(G_last - G_i)
   pdl_launch_dependents();
   pdl_wait();
   int r, c;
@@ -245,6 +245,7 @@ delta_prepare_kernel(const DeltaParams<T> p) {
       x += carried;
       carried = __shfl_sync(0xffffffffu, x, 31);
       s_g[i] = x;
+      s_up[i] = expf(x);
       s_beta[i] = i < n ? dr_sigmoid(to_float(p.b[t * p.gate_stride + h])) : 0.f;
     }
   }
@@ -284,23 +285,24 @@ delta_prepare_kernel(const DeltaParams<T> p) {
       }
   }
   const float end = s_g[DELTA_CHUNK - 1];
+  if (tid < DELTA_CHUNK) s_down[tid] = expf(end - s_g[tid]);
+  __syncthreads();
   float* w = p.w + place * DELTA_CHUNK * dp;
   float* kd = p.kd + place * DELTA_CHUNK * dp;
   float* qd = p.qd + place * DELTA_CHUNK * dp;
   for (int e = tid; e < DELTA_CHUNK * dp; e += DELTA_THREADS) {
     const int i = e / dp, d = e % dp;
-    kd[e] = kn[i * ds + d] * expf(end - s_g[i]);
-    qd[e] = qn[i * ds + d] * expf(s_g[i]);
+    kd[e] = kn[i * ds + d] * s_down[i];
+    qd[e] = qn[i * ds + d] * s_up[i];
   }
-  if (tid == 0) p.decay[place] = expf(end);
-  __syncthreads();
+  if (tid == 0) p.decay[place] = s_up[DELTA_CHUNK - 1];
   // forward substitution, a thread per column of [K | V]
   float* u = p.u + place * DELTA_CHUNK * p.v_pad;
   for (int column = tid; column < dp + p.v_pad; column += DELTA_THREADS) {
     float x[DELTA_CHUNK];
     if (column < dp) {
 #pragma unroll
-      for (int i = 0; i < DELTA_CHUNK; i++) x[i] = s_beta[i] * expf(s_g[i]) * kn[i * ds + column];
+      for (int i = 0; i < DELTA_CHUNK; i++) x[i] = s_beta[i] * s_up[i] * kn[i * ds + column];
     } else {
       const int vc = column - dp;
       const T* src = p.v + (size_t)first * p.stride + (size_t)h * p.vdim + vc;
@@ -331,10 +333,10 @@ __global__ void __launch_bounds__(DELTA_THREADS)
 delta_carry_kernel(const DeltaParams<T> p, int buffers) {
   extern __shared__ float4 carry_smem[];
   const int dim = p.dim, dp = p.dim_pad, ds = dp + 4, vp = p.v_pad, vdim = p.vdim;
-  float* S = reinterpret_cast<float*>(carry_smem);        // [dp][16]
-  float* us = S + dp * CARRY_COLS;                        // [64][16]
-  float* part = us + DELTA_CHUNK * CARRY_COLS;            // [4][64][16], or the second half's sums [dp][16]
-  const int part_floats = max(4 * DELTA_CHUNK * CARRY_COLS, dp * CARRY_COLS);
+  float* S = reinterpret_cast<float*>(carry_smem);        // [dp][20], 16 columns used
+  float* us = S + dp * CARRY_STRIDE;                      // [64][16]
+  float* part = us + DELTA_CHUNK * CARRY_COLS;            // [4][64][20], or the second half's sums [dp][20]
+  const int part_floats = max(4 * DELTA_CHUNK, dp) * CARRY_STRIDE;
   float* tiles = part + part_floats;                      // per buffer W [64][ds], keys [64][dp]
   const int tile_floats = DELTA_CHUNK * (ds + dp);
   pdl_launch_dependents();
@@ -352,7 +354,7 @@ delta_carry_kernel(const DeltaParams<T> p, int buffers) {
   float* mine = p.state + (((size_t)slot * p.heads + h) * dim) * vdim;
   for (int e = tid; e < dp * CARRY_COLS; e += DELTA_THREADS) {
     const int d = e / CARRY_COLS, c = col0 + e % CARRY_COLS;
-    S[e] = d < dim && c < vdim ? mine[(size_t)d * vdim + c] : 0.f;
+    S[d * CARRY_STRIDE + e % CARRY_COLS] = d < dim && c < vdim ? mine[(size_t)d * vdim + c] : 0.f;
   }
   auto load = [&](int c, int buf) {
     const size_t place = (size_t)(base + c) * p.heads + h;
@@ -369,8 +371,22 @@ delta_carry_kernel(const DeltaParams<T> p, int buffers) {
   };
   load(0, 0);
   dr_cp_commit();
+  // the thread's part of U0 and the chunk's decay, fetched a chunk ahead
+  const int ui = tid >> 2, uc = (tid & 3) * 4;
+  const bool u_there = col0 + uc < vp;
+  auto u_at = [&](int c) {
+    return reinterpret_cast<float4*>(p.u + ((size_t)(base + c) * p.heads + h) * DELTA_CHUNK * vp + (size_t)ui * vp + col0 + uc);
+  };
+  float4 next_u = u_there ? *u_at(0) : make_float4(0.f, 0.f, 0.f, 0.f);
+  float next_decay = p.decay[(size_t)base * p.heads + h];
   for (int c = 0; c < chunks; c++) {
     const int buf = buffers == 2 ? c & 1 : 0;
+    float4 own = next_u;
+    const float decay = next_decay;
+    if (c + 1 < chunks) {
+      if (u_there) next_u = *u_at(c + 1);
+      next_decay = p.decay[(size_t)(base + c + 1) * p.heads + h];
+    }
     if (buffers == 2 && c + 1 < chunks) {
       load(c + 1, buf ^ 1);
       dr_cp_commit();
@@ -391,7 +407,7 @@ delta_carry_kernel(const DeltaParams<T> p, int buffers) {
       for (int d = ks * 4; d < dp; d += 16) {
         float4 s[4];
 #pragma unroll
-        for (int e = 0; e < 4; e++) s[e] = *reinterpret_cast<const float4*>(S + (d + e) * CARRY_COLS + ct * 4);
+        for (int e = 0; e < 4; e++) s[e] = *reinterpret_cast<const float4*>(S + (d + e) * CARRY_STRIDE + ct * 4);
 #pragma unroll
         for (int a = 0; a < 4; a++) {
           const float4 x = *reinterpret_cast<const float4*>(tw + (rt + 16 * a) * ds + d);
@@ -403,29 +419,24 @@ delta_carry_kernel(const DeltaParams<T> p, int buffers) {
       }
 #pragma unroll
       for (int a = 0; a < 4; a++)
-        *reinterpret_cast<float4*>(part + (ks * DELTA_CHUNK + rt + 16 * a) * CARRY_COLS + ct * 4) =
+        *reinterpret_cast<float4*>(part + (ks * DELTA_CHUNK + rt + 16 * a) * CARRY_STRIDE + ct * 4) =
             make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
     }
     __syncthreads();
     {
-      const int i = tid >> 2, c4 = (tid & 3) * 4;
-      float4 sum = make_float4(0.f, 0.f, 0.f, 0.f), own = sum;
+      float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
       for (int ks = 0; ks < 4; ks++) {
-        const float4 x = *reinterpret_cast<const float4*>(part + (ks * DELTA_CHUNK + i) * CARRY_COLS + c4);
+        const float4 x = *reinterpret_cast<const float4*>(part + (ks * DELTA_CHUNK + ui) * CARRY_STRIDE + uc);
         sum.x += x.x; sum.y += x.y; sum.z += x.z; sum.w += x.w;
       }
-      float4* u = reinterpret_cast<float4*>(p.u + place * DELTA_CHUNK * vp + (size_t)i * vp + col0 + c4);
-      const bool there = col0 + c4 < vp;
-      if (there) own = *u;
       own.x -= sum.x; own.y -= sum.y; own.z -= sum.z; own.w -= sum.w;
-      if (there) *u = own;
-      *reinterpret_cast<float4*>(us + i * CARRY_COLS + c4) = own;
+      if (u_there) *u_at(c) = own;
+      *reinterpret_cast<float4*>(us + ui * CARRY_COLS + uc) = own;
     }
     __syncthreads();
     {
       // S <- decay S + K~^T U: tiles of 4 rows x 4 columns of S, the chunk's tokens in two halves
-      const float decay = p.decay[place];
       float* before = p.before + place * dp * vp;
       const int half = tid >> 7;
       for (int tile0 = 0; tile0 < dp; tile0 += 128) {
@@ -448,15 +459,15 @@ delta_carry_kernel(const DeltaParams<T> p, int buffers) {
           if (half == 1) {
 #pragma unroll
             for (int a = 0; a < 4; a++)
-              *reinterpret_cast<float4*>(part + (d0 + a) * CARRY_COLS + ct * 4) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
+              *reinterpret_cast<float4*>(part + (d0 + a) * CARRY_STRIDE + ct * 4) = make_float4(acc[a][0], acc[a][1], acc[a][2], acc[a][3]);
           }
         }
         __syncthreads();
         if (there && half == 0) {
 #pragma unroll
           for (int a = 0; a < 4; a++) {
-            float4* at = reinterpret_cast<float4*>(S + (d0 + a) * CARRY_COLS + ct * 4);
-            const float4 s = *at, more = *reinterpret_cast<const float4*>(part + (d0 + a) * CARRY_COLS + ct * 4);
+            float4* at = reinterpret_cast<float4*>(S + (d0 + a) * CARRY_STRIDE + ct * 4);
+            const float4 s = *at, more = *reinterpret_cast<const float4*>(part + (d0 + a) * CARRY_STRIDE + ct * 4);
             if (col0 + ct * 4 < vp) *reinterpret_cast<float4*>(before + (size_t)(d0 + a) * vp + col0 + ct * 4) = s;
             *at = make_float4(fmaf(decay, s.x, acc[a][0] + more.x), fmaf(decay, s.y, acc[a][1] + more.y),
                               fmaf(decay, s.z, acc[a][2] + more.z), fmaf(decay, s.w, acc[a][3] + more.w));
@@ -473,7 +484,7 @@ delta_carry_kernel(const DeltaParams<T> p, int buffers) {
   __syncthreads();
   for (int e = tid; e < dp * CARRY_COLS; e += DELTA_THREADS) {
     const int d = e / CARRY_COLS, c = col0 + e % CARRY_COLS;
-    if (d < dim && c < vdim) mine[(size_t)d * vdim + c] = S[e];
+    if (d < dim && c < vdim) mine[(size_t)d * vdim + c] = S[d * CARRY_STRIDE + e % CARRY_COLS];
   }
 }
 
@@ -565,7 +576,7 @@ constexpr int DELTA_MAX_SMEM = 227 * 1024 - 1024;
 size_t prepare_bytes(int dp) { return (size_t)(2 * DELTA_CHUNK * (dp + 4) + DELTA_CHUNK * PREP_A_STRIDE) * sizeof(float); }
 size_t carry_bytes(int dp, int buffers) {
   const int part = 4 * DELTA_CHUNK > dp ? 4 * DELTA_CHUNK : dp;
-  return (size_t)((dp + DELTA_CHUNK + part) * CARRY_COLS + buffers * DELTA_CHUNK * (2 * dp + 4)) * sizeof(float);
+  return (size_t)((dp + part) * CARRY_STRIDE + DELTA_CHUNK * CARRY_COLS + buffers * DELTA_CHUNK * (2 * dp + 4)) * sizeof(float);
 }
 size_t outputs_bytes(int dp) {
   return (size_t)(DELTA_CHUNK * (dp + 4) + dp * OUT_COLS + DELTA_CHUNK * PREP_A_STRIDE + DELTA_CHUNK * OUT_COLS) * sizeof(float);
