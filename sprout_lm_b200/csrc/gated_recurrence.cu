@@ -56,7 +56,7 @@ struct ScanParams {
   float* sums;                         // [max_chunks, heads, dim, vdim]: a chunk's own sums, then the state before the chunk
   float* prods;                        // [max_chunks, heads, dim]: the product of a chunk's decays
   int chunk, requests;
-  int q_silu;                          // silu on the query rows
+  int q_silu;                          // silu on the query rows (with a floor only)
   int v_cols, ones_col;                // columns the value rows really have (<= vdim); column v_cols of the state is fed 1
 };
 
@@ -92,7 +92,8 @@ constexpr int SCAN_THREADS = 128, SCAN_MAX_TOKENS = 8;
 // request's state.  The decays of these two walks are made beforehand by scan_decay_kernel (each is needed by all
 // blocks of columns and in both walks).  Against the single walk only the association of the decays' products
 // differs: (a_n ... a_1) S + sums instead of a_n (... (a_1 S)).
-template <typename T, int ROWS, int COLS, int PHASE>
+// FLOOR: the forget gate with a floor (DECAY_FLOOR); a form of its own, so that the others keep their registers.
+template <typename T, int ROWS, int COLS, int PHASE, bool FLOOR>
 __global__ void __launch_bounds__(SCAN_THREADS, ROWS == 8 ? 4 : 2)
 gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
   constexpr int ROWS_LOG2 = ROWS == 8 ? 3 : 5;
@@ -123,8 +124,8 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
     return;
   }
   const int g = h / (p.heads / p.groups);
-  const bool floored = p.mode == DECAY_FLOOR;         // a decay per channel, and no keys
-  const bool per_head = p.mode != DECAY_PER_CHANNEL && !floored;
+  constexpr bool floored = FLOOR;                     // a decay per channel, and no keys
+  const bool per_head = !FLOOR && p.mode != DECAY_PER_CHANNEL;
   float* mine = p.state + (((size_t)slot * p.heads + h) * dim) * p.vdim;
   // the chunk's place in the scratch: the blocks before it belong to the requests before r and to r's earlier chunks
   float* held = PHASE == SCAN_WHOLE ? nullptr : p.sums + (((size_t)(blockIdx.x) * p.heads + h) * dim) * p.vdim;
@@ -206,7 +207,7 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
         } else {
           decay = expf(-softplus_f(-(rz[u] + p.bias[(size_t)h * dim + i])) * p.inv_tau);  // sigmoid(z)^(1/tau) through its logarithm
         }
-        x.x = (p.q_silu ? silu_g(rq[u]) : rq[u]) * p.q_scale;
+        x.x = (FLOOR && p.q_silu ? silu_g(rq[u]) : rq[u]) * p.q_scale;
         x.y = floored ? decay : rk[u] * step;
         x.z = floored ? 1.0f - decay : decay;
       }
@@ -456,7 +457,7 @@ __global__ void scaled_sum_kernel(float* __restrict__ x, const float* __restrict
     x[i] += a * y1[i] + (y2 ? b * y2[i] : 0.f);
 }
 
-template <typename T, int ROWS, int COLS>
+template <typename T, int ROWS, int COLS, bool FLOOR>
 int launch_scan_tiles(const ScanParams<T>& p, int requests, int max_chunks, cudaStream_t stream) {
   int slices_log2 = 0;
   while ((ROWS << slices_log2) < p.dim) slices_log2++;
@@ -472,30 +473,31 @@ int launch_scan_tiles(const ScanParams<T>& p, int requests, int max_chunks, cuda
   const dim3 grid(requests, p.heads, (p.vdim + cb - 1) / cb);
   SPROUT_REQUIRE(grid.z <= 65535, "gated_scan: too many value columns");
   if (p.sums == nullptr && p.mode == DECAY_GIVEN) {
-    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT, FLOOR>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
     return sprout_check_launch("gated_scan");
   }
   if (p.sums == nullptr) {
-    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_WHOLE>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_WHOLE, FLOOR>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
     return sprout_check_launch("gated_scan");
   }
   // `max_chunks` blocks per (head, columns): the chunks of all requests, found by their number
   const dim3 chunks(max_chunks, p.heads, grid.z);
-  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_SUMS>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_SUMS, FLOOR>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
   if (int rc = sprout_check_launch("gated_scan (chunk sums)")) return rc;
   SPROUT_REQUIRE(requests <= 65535, "gated_scan: too many requests");
   sprout_launch(scan_carry_kernel, dim3((p.dim * p.vdim + 255) / 256, p.heads, requests), dim3(256), 0, stream, p.sums,
                 (const float*)p.prods, (const float*)p.state, p.q_start, p.state_slots, p.num_slots, p.chunk, p.heads, p.dim, p.vdim);
   if (int rc = sprout_check_launch("gated_scan (carry)")) return rc;
-  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT, FLOOR>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
   return sprout_check_launch("gated_scan (chunk outputs)");
 }
 
 template <typename T>
 int launch_scan(const ScanParams<T>& p, int requests, int max_chunks, cudaStream_t stream) {
   // a thread's tile of the state: 8 rows x 4 columns up to 256 key channels, 32 rows of one column up to 1024
-  if (p.dim <= 8 * 32) return launch_scan_tiles<T, 8, 4>(p, requests, max_chunks, stream);
-  return launch_scan_tiles<T, 32, 1>(p, requests, max_chunks, stream);
+  if (p.mode == DECAY_FLOOR)
+    return p.dim <= 8 * 32 ? launch_scan_tiles<T, 8, 4, true>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, true>(p, requests, max_chunks, stream);
+  return p.dim <= 8 * 32 ? launch_scan_tiles<T, 8, 4, false>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, false>(p, requests, max_chunks, stream);
 }
 
 }  // namespace
@@ -527,6 +529,7 @@ SPROUT_API int sprout_gated_scan(const void* q, int q_stride, const void* k, int
   SPROUT_REQUIRE(requests > 0 && heads > 0 && groups > 0 && heads % groups == 0 && dim > 0 && vdim > 0 && num_slots > 0,
                  "gated_scan: bad sizes");
   SPROUT_REQUIRE(mode == DECAY_PER_CHANNEL || ((mode == DECAY_PER_HEAD || mode == DECAY_FLOOR) && a_log) || mode == DECAY_GIVEN, "gated_scan: unknown decay form");
+  SPROUT_REQUIRE(!q_silu || mode == DECAY_FLOOR, "gated_scan: silu on the queries goes with a floor");
   SPROUT_REQUIRE(mode != DECAY_FLOOR || groups == heads, "gated_scan: a forget gate with a floor has query vectors per head");
   SPROUT_REQUIRE(heads <= 65535, "gated_scan: too many heads");
   if (dtype == SPROUT_F32) {

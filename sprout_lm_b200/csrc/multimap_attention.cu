@@ -309,7 +309,7 @@ multimap_attention_simple_kernel(const T* __restrict__ q, int q_stride, const T*
   }
   float factor = out_scale;
   if (norm_eps > 0.f) factor *= 1.0f / sqrtf(block_sum(squares, scratch) / (float)vdim + norm_eps);
-  if (turn.cos != nullptr) {
+  if (MAPS == 1 && turn.cos != nullptr) {
     float* whole = (float*)(row_index + CHUNK);       // vdim
 #pragma unroll
     for (int part = 0; part < PARTS; part++)
@@ -327,8 +327,8 @@ multimap_attention_simple_kernel(const T* __restrict__ q, int q_stride, const T*
       o[part] = leads ? o[part] * c + other * s : o[part] * c - other * s;
     }
   }
-  if (gate != nullptr && !gate_elements) factor *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + h])));
-  const T* gates = gate != nullptr && gate_elements ? gate + (size_t)t * gate_stride + (size_t)h * vdim : nullptr;
+  if (gate != nullptr && !(MAPS == 1 && gate_elements)) factor *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + h])));
+  const T* gates = MAPS == 1 && gate != nullptr && gate_elements ? gate + (size_t)t * gate_stride + (size_t)h * vdim : nullptr;
   T* dst = out + (size_t)t * out_stride + (size_t)h * vdim;
 #pragma unroll
   for (int part = 0; part < PARTS; part++)
@@ -708,7 +708,7 @@ multimap_attention_mma_kernel(const MultiMapParams p) {
     f0 *= 1.0f / sqrtf(sq0 / (float)VDIM + p.norm_eps);
     f1 *= 1.0f / sqrtf(sq1 / (float)VDIM + p.norm_eps);
   }
-  if (p.turn.cos != nullptr) {
+  if (MAPS == 1 && p.turn.cos != nullptr) {
     // back by the query's position, on the accumulators: both elements of a pair are this thread's
     const size_t at0 = (size_t)min(max(limit0, 0), p.turn.positions - 1) * (VDIM / 2), at1 = (size_t)min(max(limit1, 0), p.turn.positions - 1) * (VDIM / 2);
     if (p.turn.interleaved) {
@@ -733,7 +733,7 @@ multimap_attention_mma_kernel(const MultiMapParams p) {
         }
     }
   }
-  if (p.gate != nullptr && p.gate_elements) {
+  if (MAPS == 1 && p.gate != nullptr && p.gate_elements) {
 #pragma unroll
     for (int i = 0; i < VDIM / 8; i++)
 #pragma unroll
@@ -801,7 +801,7 @@ multimap_merge_kernel(const MultiMapParams p, int vdim) {
     if (threadIdx.x + part * 128 < vdim) squares = fmaf(v[part], v[part], squares);
   float factor = p.out_scale;
   if (p.norm_eps > 0.f) factor *= 1.0f / sqrtf(block_sum(squares, scratch) / (float)vdim + p.norm_eps);
-  if (p.turn.cos != nullptr) {
+  if (MAPS == 1 && p.turn.cos != nullptr) {
 #pragma unroll
     for (int part = 0; part < 2; part++)
       if (threadIdx.x + part * 128 < vdim) whole[threadIdx.x + part * 128] = v[part];
@@ -818,7 +818,7 @@ multimap_merge_kernel(const MultiMapParams p, int vdim) {
       v[part] = leads ? v[part] * c + other * s : v[part] * c - other * s;
     }
   }
-  if (p.gate != nullptr && p.gate_elements) {
+  if (MAPS == 1 && p.gate != nullptr && p.gate_elements) {
 #pragma unroll
     for (int part = 0; part < 2; part++)
       if (threadIdx.x + part * 128 < vdim) v[part] *= element_gate(p, token, head, vdim, threadIdx.x + part * 128);
@@ -890,6 +890,7 @@ SPROUT_API int sprout_multimap_attention_mma(const void* q, int q_stride, const 
                    num_pages, scale, lambda, norm_eps, out_scale, status, ksplit, partial, mask_kind, mask_size, sink,
                    (const __nv_bfloat16*)gate, gate_stride, mask_keep, softcap, gate_elements,
                    {turn_cos, turn_sin, turn_positions, turn_interleaved}};
+  SPROUT_REQUIRE(maps == 1 || (!turn_cos && !gate_elements), "multimap_attention_mma: turned values and element gates are for one map per head");
   SPROUT_REQUIRE(!turn_cos || (turn_sin && turn_positions > 0), "multimap_attention_mma: the turn's tables are missing");
   SPROUT_REQUIRE(mask_kind == MASK_CAUSAL || ((mask_kind == MASK_WINDOW || mask_kind == MASK_CHUNK) && mask_size > 0),
                  "multimap_attention_mma: a window or a chunk needs a positive size");
@@ -965,6 +966,7 @@ SPROUT_API int sprout_multimap_attention_simple(const void* q, int q_stride, con
   SPROUT_REQUIRE(mask_kind == MASK_CAUSAL || ((mask_kind == MASK_WINDOW || mask_kind == MASK_CHUNK) && mask_size > 0),
                  "multimap_attention: a window or a chunk needs a positive size");
   SPROUT_REQUIRE(!gate || gate_stride >= (gate_elements ? heads * vdim : heads), "multimap_attention: gate rows hold a number per head or element");
+  SPROUT_REQUIRE(maps == 1 || (!turn_cos && !gate_elements), "multimap_attention: turned values and element gates are for one map per head");
   SPROUT_REQUIRE(!turn_cos || (turn_sin && turn_positions > 0 && vdim % 2 == 0), "multimap_attention: the turn's tables are missing");
   const OutputTurn turn{turn_cos, turn_sin, turn_positions, turn_interleaved};
   SPROUT_REQUIRE(mask_keep >= 0 && (mask_keep == 0 || mask_kind == MASK_WINDOW) && softcap >= 0.f,

@@ -1557,7 +1557,7 @@ def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: 
     stride of one dtype.  Per key channel (default): z [tokens, heads * dim] (of that dtype or float32), a = sigmoid(z + bias)^(1 / tau), c = 1.
     ``per_head``: z [tokens, heads], dt = softplus(z + bias), a = exp(-exp(a_log) dt) for all of the head's channels, c = dt.
     ``floor`` (float32 [heads * dim]): z [tokens, heads * dim], a = floor + (1 - floor) sigmoid(z + bias) and 1 - a takes the place
-    of c k (``k`` is None).  ``q_silu``: q passes silu first.
+    of c k (``k`` is None); with ``q_silu`` q passes silu first (in this form only).
     ``given`` = (a, c), float32 [tokens, heads] each: the decay and the factor on k per head, ready-made (z and bias are None).
     ``ones_col``: the value rows are narrower than the state, v [tokens, heads * v_cols] with v_cols < vdim, and the state's
     column v_cols is fed the constant 1 as a value (the columns after it 0): that column of the state is then the sum of the
