@@ -213,7 +213,7 @@ def test_a_lost_state_a_dropped_sink_or_a_shifted_window_shows(tmp_path):
             return moved(plain.forward(config, tensors, tokens))
         finally:
             setattr(plain, key, real[key])
-    print("planted", planted("rotate", lambda x, p, b, d, i: x if (np.asarray(p) < 0).any() else real["rotate"](x, p, b, d, i)))      # no turn back
+    assert planted("rotate", lambda x, p, b, d, i: x if (np.asarray(p) < 0).any() else real["rotate"](x, p, b, d, i)) > bar      # no turn back
     assert planted("softmax_attention", lambda *a, window=None, unit_sink=False: real["softmax_attention"](*a, window=window)) > bar
     assert planted("delta_rule", lambda q, k, v, g, beta: real["delta_rule"](q, 0 * k + k, v, np.ones_like(g), beta)) > bar
     assert planted("forget_and_write", lambda q, f, v: real["forget_and_write"](q, np.minimum(f, 0.9), v)) > bar
