@@ -9,6 +9,9 @@
 //                                                             c_t = dt;
 //                    a floor (a forget gate that also decides what is written): w_t[i] = (1 - floor[i]) sigmoid(-(z_t[i] + bias[i])),
 //                                                             a_t[i] = 1 - w_t[i]; w_t takes the place of c_t k_t;
+//                    a bonus (the RWKV recurrence): a_t[i] = exp(-exp(z_t[i] + bias[i])), c_t = 1, and the output reads the state before
+//                                                             the token plus the token's own write weighed by a bonus u[i] per channel:
+//                                                             o_t = (S_(t-1) + diag(u) k_t v_t^T)^T (q_scale q_t);
 //                    given (a matrix memory with exponential gates): a_t and c_t per head come ready-made from the
 //                                                             caller (`da`, `dc`), whatever the portion's length.
 //                  With `ones_col` the value row gets one more column that is always 1 (column `v_cols` of the state
@@ -20,6 +23,8 @@
 //  * causal_conv:  y_t[c] = act(bias[c] + sum_j w[c][j] x_(t - (taps - 1 - j))[c]), zeros before the start of the
 //                  sequence; the last taps - 1 inputs of a request live in its state slot [taps - 1, channels] and are
 //                  read at the start of a portion and replaced at its end.
+//  * token_blend:  row t of part s = h_t + (h_(t-1) - h_t) * mu_s, several blends of every row with the row before it; the row
+//                  before a portion's first lives in the request's state slot (zeros at the start of the sequence).
 //  * gated_group_norm: rows in `groups` equal parts, each divided by its own root mean square, times a weight that
 //                  repeats every `period` elements, times act(gate) before or after the norm (or without a gate).
 //  * scaled_sum:   x += a y_1 + b y_2.
@@ -31,7 +36,11 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + lo
 __device__ __forceinline__ float silu_g(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_g(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-enum ScanDecay : int { DECAY_PER_CHANNEL = 0, DECAY_PER_HEAD = 1, DECAY_GIVEN = 2, DECAY_FLOOR = 3 };
+enum ScanDecay : int { DECAY_PER_CHANNEL = 0, DECAY_PER_HEAD = 1, DECAY_GIVEN = 2, DECAY_FLOOR = 3, DECAY_BONUS = 4 };
+// Forms of the scan's kernel (the others share FORM_PLAIN), so that each keeps its own registers.
+enum ScanForm : int { FORM_PLAIN = 0, FORM_FLOOR = 1, FORM_BONUS = 2 };
+
+__device__ __forceinline__ float double_exp_decay(float z) { return expf(-expf(z)); }
 
 // What a forget gate with a floor writes: 1 - f for f = floor + (1 - floor) sigmoid(z).
 __device__ __forceinline__ float write_share(float z, float floor) { return (1.0f - floor) * sigmoid_g(-z); }
@@ -45,6 +54,7 @@ struct ScanParams {
   const float* bias;                   // added to z: [heads * dim] or [heads]
   const float* a_log;                  // per head (per-head decay only); with a floor: the floors [heads * dim]
   const float* skip;                   // per head, or null
+  const float* bonus;                  // [heads * dim] (DECAY_BONUS only)
   float inv_tau, q_scale;
   int mode, heads, groups, dim, vdim;
   const int* q_start; const int* state_slots; float* state; int num_slots;
@@ -92,8 +102,9 @@ constexpr int SCAN_THREADS = 128, SCAN_MAX_TOKENS = 8;
 // request's state.  The decays of these two walks are made beforehand by scan_decay_kernel (each is needed by all
 // blocks of columns and in both walks).  Against the single walk only the association of the decays' products
 // differs: (a_n ... a_1) S + sums instead of a_n (... (a_1 S)).
-// FLOOR: the forget gate with a floor (DECAY_FLOOR); a form of its own, so that the others keep their registers.
-template <typename T, int ROWS, int COLS, int PHASE, bool FLOOR>
+// FORM: FORM_FLOOR is the forget gate with a floor (DECAY_FLOOR), FORM_BONUS the output that reads the state before the token
+// (DECAY_BONUS): the fourth number of a row's vector is then q_scale q u k, whose sum over the rows weighs the token's value.
+template <typename T, int ROWS, int COLS, int PHASE, int FORM>
 __global__ void __launch_bounds__(SCAN_THREADS, ROWS == 8 ? 4 : 2)
 gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
   constexpr int ROWS_LOG2 = ROWS == 8 ? 3 : 5;
@@ -124,8 +135,8 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
     return;
   }
   const int g = h / (p.heads / p.groups);
-  constexpr bool floored = FLOOR;                     // a decay per channel, and no keys
-  const bool per_head = !FLOOR && p.mode != DECAY_PER_CHANNEL;
+  constexpr bool floored = FORM == FORM_FLOOR, bonus = FORM == FORM_BONUS;                     // a decay per channel, and no keys
+  const bool per_head = FORM == FORM_PLAIN && p.mode != DECAY_PER_CHANNEL;
   float* mine = p.state + (((size_t)slot * p.heads + h) * dim) * p.vdim;
   // the chunk's place in the scratch: the blocks before it belong to the requests before r and to r's earlier chunks
   float* held = PHASE == SCAN_WHOLE ? nullptr : p.sums + (((size_t)(blockIdx.x) * p.heads + h) * dim) * p.vdim;
@@ -204,12 +215,15 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
           decay = expf(-rate * step);
         } else if (floored) {
           decay = write_share(rz[u] + p.bias[(size_t)h * dim + i], p.a_log[(size_t)h * dim + i]);
+        } else if (bonus) {
+          decay = double_exp_decay(rz[u] + p.bias[(size_t)h * dim + i]);
         } else {
           decay = expf(-softplus_f(-(rz[u] + p.bias[(size_t)h * dim + i])) * p.inv_tau);  // sigmoid(z)^(1/tau) through its logarithm
         }
-        x.x = (FLOOR && p.q_silu ? silu_g(rq[u]) : rq[u]) * p.q_scale;
+        x.x = (floored && p.q_silu ? silu_g(rq[u]) : rq[u]) * p.q_scale;
         x.y = floored ? decay : rk[u] * step;
         x.z = floored ? 1.0f - decay : decay;
+        if (bonus && PHASE != SCAN_CHUNK_SUMS) x.w = x.x * p.bonus[(size_t)h * dim + i] * x.y;
       }
       tok[e] = x;
     }
@@ -233,18 +247,24 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
 #pragma unroll
       for (int c = 0; c < COLS; c++) o[c] = 0.f;
       const float4* cur = tok + ((size_t)tt << rows_log2) + slice;
+      float own = 0.f;                                 // the weight of the token's own value
 #pragma unroll
       for (int j = 0; j < ROWS; j++) {
         const float4 x = cur[j << slices_log2];
 #pragma unroll
         for (int c = 0; c < COLS; c++) {
           const float s = fmaf(x.z, S[j][c], x.y * v[c]);
+          if (PHASE != SCAN_CHUNK_SUMS) o[c] = fmaf(bonus ? S[j][c] : s, x.x, o[c]);
           S[j][c] = s;
-          if (PHASE != SCAN_CHUNK_SUMS) o[c] = fmaf(s, x.x, o[c]);
         }
+        if (bonus && PHASE != SCAN_CHUNK_SUMS) own += x.w;
         if (PHASE == SCAN_CHUNK_SUMS) P[j] *= x.z;
       }
       if (PHASE == SCAN_CHUNK_SUMS) continue;
+      if (bonus) {
+#pragma unroll
+        for (int c = 0; c < COLS; c++) o[c] = fmaf(own, v[c], o[c]);
+      }
       float* dst = out_rows + tt * p.heads * p.vdim;
       if (COLS == 4 && slices_log2 >= 2) {
         // four sums over the slices with five shuffles instead of four per sum: neighbours split the columns between
@@ -288,7 +308,8 @@ gated_scan_kernel(const ScanParams<T> p, int slices_log2, int batch) {
 }
 
 // The decays of every token of the step, once: per key channel a = sigmoid(z + bias)^(1 / tau); per head
-// dt = softplus(z + bias), a = exp(-exp(a_log) dt), c = dt; with a floor what is written, 1 - a (`a_log` holds the floors).
+// dt = softplus(z + bias), a = exp(-exp(a_log) dt), c = dt; with a floor what is written, 1 - a (`a_log` holds the floors);
+// with a bonus a = exp(-exp(z + bias)).
 __global__ void scan_decay_kernel(const void* __restrict__ z, int z_stride, int z_f32, int is_bf16, const float* __restrict__ bias,
                                   const float* __restrict__ a_log, float inv_tau, int mode, int heads, int dim, long long count,
                                   float* __restrict__ da, float* __restrict__ dc) {
@@ -306,6 +327,8 @@ __global__ void scan_decay_kernel(const void* __restrict__ z, int z_stride, int 
       dc[e] = step;
     } else if (mode == DECAY_FLOOR) {
       da[e] = write_share(zv + bias[c], a_log[c]);
+    } else if (mode == DECAY_BONUS) {
+      da[e] = double_exp_decay(zv + bias[c]);
     } else {
       da[e] = expf(-softplus_f(-(zv + bias[c])) * inv_tau);
     }
@@ -419,17 +442,87 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
   }
 }
 
-// grid (rows, groups).  o float32 [rows, width]; gate rows of T with their own stride; out rows of T.
-template <typename T>
+// A thread takes VEC neighbouring elements of one row in every part.  The thread of a portion's first token reads the row before
+// it from the request's state and then puts the request's last row there (no other thread touches that element).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+token_blend_kernel(const T* __restrict__ h, const float* __restrict__ mu, T* __restrict__ out, const int* __restrict__ q_start,
+                   const int* __restrict__ seq_of_token, const int* __restrict__ state_slots, float* __restrict__ state, int num_slots,
+                   int tokens, int width, int parts, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int per_row = width / VEC;
+  const long long count = (long long)tokens * per_row;
+  for (long long e = blockIdx.x * (long long)blockDim.x + threadIdx.x; e < count; e += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(e / per_row), c = (int)(e - (long long)t * per_row) * VEC;
+    const int r = seq_of_token[t], begin = q_start[r];
+    float now[VEC], delta[VEC];
+    auto row = [&](int token, float (&v)[VEC]) {
+      const T* src = h + (size_t)token * width + c;
+      if (VEC == 8 && sizeof(T) == 2) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(src);
+        const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < VEC / 2; i++) {
+          const float2 f = __bfloat1622float2(pairs[i]);
+          v[2 * i] = f.x; v[2 * i + 1] = f.y;
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; i++) v[i] = to_float(src[i]);
+      }
+    };
+    row(t, now);
+    if (t > begin) {
+      row(t - 1, delta);
+    } else {
+      const int slot = state_slots[r];
+      if (slot < 0 || slot >= num_slots) {
+        if (c == 0) atomicOr(status, SPROUT_STATUS_BAD_PAGE);
+#pragma unroll
+        for (int i = 0; i < VEC; i++) delta[i] = 0.f;
+      } else {
+        float* mine = state + (size_t)slot * width + c;
+        float last[VEC];
+        row(q_start[r + 1] - 1, last);
+#pragma unroll
+        for (int i = 0; i < VEC; i++) {
+          delta[i] = mine[i];
+          mine[i] = last[i];
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; i++) delta[i] -= now[i];
+    for (int s = 0; s < parts; s++) {
+      const float* m = mu + (size_t)s * width + c;
+      T* dst = out + ((size_t)t * parts + s) * width + c;
+      if (VEC == 8 && sizeof(T) == 2) {
+        uint4 packed;
+        __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+        for (int i = 0; i < VEC / 2; i++)
+          pairs[i] = __floats2bfloat162_rn(fmaf(delta[2 * i], m[2 * i], now[2 * i]), fmaf(delta[2 * i + 1], m[2 * i + 1], now[2 * i + 1]));
+        *reinterpret_cast<uint4*>(dst) = packed;
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; i++) dst[i] = from_float<T>(fmaf(delta[i], m[i], now[i]));
+      }
+    }
+  }
+}
+
+// grid (rows, groups).  o float32 [rows, width]; gate rows of TG with their own stride; out rows of T.
+template <typename TG, typename T>
 __global__ void __launch_bounds__(128)
-gated_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_stride, const float* __restrict__ weight,
+gated_group_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int gate_stride, const float* __restrict__ weight,
                         int period, T* __restrict__ out, int width, int groups, float eps, int gate_first, int act) {
   __shared__ float scratch[33];
   pdl_launch_dependents();
   pdl_wait();
   const int part = width / groups, base = blockIdx.y * part;
   const float* src = o + (size_t)blockIdx.x * width + base;
-  const T* grow = gate ? gate + (size_t)blockIdx.x * gate_stride + base : nullptr;
+  const TG* grow = gate ? gate + (size_t)blockIdx.x * gate_stride + base : nullptr;
   float q = 0.f;
   for (int i = threadIdx.x; i < part; i += blockDim.x) {
     float v = src[i];
@@ -457,7 +550,7 @@ __global__ void scaled_sum_kernel(float* __restrict__ x, const float* __restrict
     x[i] += a * y1[i] + (y2 ? b * y2[i] : 0.f);
 }
 
-template <typename T, int ROWS, int COLS, bool FLOOR>
+template <typename T, int ROWS, int COLS, int FORM>
 int launch_scan_tiles(const ScanParams<T>& p, int requests, int max_chunks, cudaStream_t stream) {
   int slices_log2 = 0;
   while ((ROWS << slices_log2) < p.dim) slices_log2++;
@@ -473,37 +566,40 @@ int launch_scan_tiles(const ScanParams<T>& p, int requests, int max_chunks, cuda
   const dim3 grid(requests, p.heads, (p.vdim + cb - 1) / cb);
   SPROUT_REQUIRE(grid.z <= 65535, "gated_scan: too many value columns");
   if (p.sums == nullptr && p.mode == DECAY_GIVEN) {
-    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT, FLOOR>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT, FORM>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
     return sprout_check_launch("gated_scan");
   }
   if (p.sums == nullptr) {
-    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_WHOLE, FLOOR>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+    sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_WHOLE, FORM>, grid, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
     return sprout_check_launch("gated_scan");
   }
   // `max_chunks` blocks per (head, columns): the chunks of all requests, found by their number
   const dim3 chunks(max_chunks, p.heads, grid.z);
-  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_SUMS, FLOOR>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_SUMS, FORM>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
   if (int rc = sprout_check_launch("gated_scan (chunk sums)")) return rc;
   SPROUT_REQUIRE(requests <= 65535, "gated_scan: too many requests");
   sprout_launch(scan_carry_kernel, dim3((p.dim * p.vdim + 255) / 256, p.heads, requests), dim3(256), 0, stream, p.sums,
                 (const float*)p.prods, (const float*)p.state, p.q_start, p.state_slots, p.num_slots, p.chunk, p.heads, p.dim, p.vdim);
   if (int rc = sprout_check_launch("gated_scan (carry)")) return rc;
-  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT, FLOOR>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
+  sprout_launch(gated_scan_kernel<T, ROWS, COLS, SCAN_CHUNK_OUT, FORM>, chunks, dim3(SCAN_THREADS), smem, stream, p, slices_log2, batch);
   return sprout_check_launch("gated_scan (chunk outputs)");
 }
 
 template <typename T>
 int launch_scan(const ScanParams<T>& p, int requests, int max_chunks, cudaStream_t stream) {
   // a thread's tile of the state: 8 rows x 4 columns up to 256 key channels, 32 rows of one column up to 1024
+  const bool narrow = p.dim <= 8 * 32;
   if (p.mode == DECAY_FLOOR)
-    return p.dim <= 8 * 32 ? launch_scan_tiles<T, 8, 4, true>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, true>(p, requests, max_chunks, stream);
-  return p.dim <= 8 * 32 ? launch_scan_tiles<T, 8, 4, false>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, false>(p, requests, max_chunks, stream);
+    return narrow ? launch_scan_tiles<T, 8, 4, FORM_FLOOR>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, FORM_FLOOR>(p, requests, max_chunks, stream);
+  if (p.mode == DECAY_BONUS)
+    return narrow ? launch_scan_tiles<T, 8, 4, FORM_BONUS>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, FORM_BONUS>(p, requests, max_chunks, stream);
+  return narrow ? launch_scan_tiles<T, 8, 4, FORM_PLAIN>(p, requests, max_chunks, stream) : launch_scan_tiles<T, 32, 1, FORM_PLAIN>(p, requests, max_chunks, stream);
 }
 
 }  // namespace
 
 SPROUT_API int sprout_gated_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
-                                 const void* z, int z_stride, int z_f32, int dtype, const float* bias, const float* a_log, const float* skip,
+                                 const void* z, int z_stride, int z_f32, int dtype, const float* bias, const float* a_log, const float* skip, const float* bonus,
                                  float inv_tau, float q_scale, int mode, int requests, int heads, int groups, int dim, int vdim,
                                  const int* q_start, const int* state_slots, float* state, int num_slots, float* out, int* status,
                                  int tokens, int chunk, int max_chunks, float* da, float* dc, float* sums, float* prods,
@@ -528,19 +624,20 @@ SPROUT_API int sprout_gated_scan(const void* q, int q_stride, const void* k, int
   }
   SPROUT_REQUIRE(requests > 0 && heads > 0 && groups > 0 && heads % groups == 0 && dim > 0 && vdim > 0 && num_slots > 0,
                  "gated_scan: bad sizes");
-  SPROUT_REQUIRE(mode == DECAY_PER_CHANNEL || ((mode == DECAY_PER_HEAD || mode == DECAY_FLOOR) && a_log) || mode == DECAY_GIVEN, "gated_scan: unknown decay form");
+  SPROUT_REQUIRE(mode == DECAY_PER_CHANNEL || ((mode == DECAY_PER_HEAD || mode == DECAY_FLOOR) && a_log) || mode == DECAY_GIVEN ||
+                 (mode == DECAY_BONUS && bonus), "gated_scan: unknown decay form");
   SPROUT_REQUIRE(!q_silu || mode == DECAY_FLOOR, "gated_scan: silu on the queries goes with a floor");
-  SPROUT_REQUIRE(mode != DECAY_FLOOR || groups == heads, "gated_scan: a forget gate with a floor has query vectors per head");
+  SPROUT_REQUIRE((mode != DECAY_FLOOR && mode != DECAY_BONUS) || groups == heads, "gated_scan: a forget gate with a floor or a bonus has query vectors per head");
   SPROUT_REQUIRE(heads <= 65535, "gated_scan: too many heads");
   if (dtype == SPROUT_F32) {
     ScanParams<float> p{(const float*)q, q_stride, (const float*)k, k_stride, (const float*)v, v_stride, z, z_stride, z_f32,
-                        bias, a_log, skip, inv_tau, q_scale, mode, heads, groups, dim, vdim, q_start, state_slots, state,
+                        bias, a_log, skip, bonus, inv_tau, q_scale, mode, heads, groups, dim, vdim, q_start, state_slots, state,
                         num_slots, out, status, da, dc, sums, prods, chunk, requests, q_silu, v_cols, ones_col};
     return launch_scan(p, requests, max_chunks, stream);
   }
   if (dtype == SPROUT_BF16) {
     ScanParams<__nv_bfloat16> p{(const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k, k_stride, (const __nv_bfloat16*)v,
-                                v_stride, z, z_stride, z_f32, bias, a_log, skip, inv_tau, q_scale, mode, heads,
+                                v_stride, z, z_stride, z_f32, bias, a_log, skip, bonus, inv_tau, q_scale, mode, heads,
                                 groups, dim, vdim, q_start, state_slots, state, num_slots, out, status, da, dc, sums, prods, chunk,
                                 requests, q_silu, v_cols, ones_col};
     return launch_scan(p, requests, max_chunks, stream);
@@ -569,17 +666,45 @@ SPROUT_API int sprout_causal_conv(const void* in, int in_stride, const float* we
   return sprout_check_launch("causal_conv");
 }
 
-SPROUT_API int sprout_gated_group_norm(const float* o, const void* gate, int gate_stride, const float* weight, int period, void* out,
+// out [tokens, parts, width]: row t of part s = h_t + (h_(t-1) - h_t) * mu[s]; state float32 [slots, width], the last row of
+// every request.
+SPROUT_API int sprout_token_blend(const void* h, const float* mu, void* out, int dtype, const int* q_start, const int* seq_of_token,
+                                  const int* state_slots, float* state, int num_slots, int tokens, int width, int parts, int* status,
+                                  cudaStream_t stream) {
+  SPROUT_REQUIRE(h && mu && out && q_start && seq_of_token && state_slots && state && status, "token_blend: null pointer");
+  SPROUT_REQUIRE(tokens > 0 && width > 0 && parts > 0 && num_slots > 0, "token_blend: bad sizes");
+  const bool vec = dtype == SPROUT_BF16 && width % 8 == 0 && (((uintptr_t)h | (uintptr_t)out) & 15) == 0;
+  const long long blocks = ((long long)tokens * (width / (vec ? 8 : 1)) + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
+  if (dtype == SPROUT_F32)
+    sprout_launch(token_blend_kernel<float, 1>, grid, dim3(256), 0, stream, (const float*)h, mu, (float*)out, q_start, seq_of_token,
+                  state_slots, state, num_slots, tokens, width, parts, status);
+  else if (vec)
+    sprout_launch(token_blend_kernel<__nv_bfloat16, 8>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)h, mu, (__nv_bfloat16*)out,
+                  q_start, seq_of_token, state_slots, state, num_slots, tokens, width, parts, status);
+  else if (dtype == SPROUT_BF16)
+    sprout_launch(token_blend_kernel<__nv_bfloat16, 1>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)h, mu, (__nv_bfloat16*)out,
+                  q_start, seq_of_token, state_slots, state, num_slots, tokens, width, parts, status);
+  else
+    return sprout_fail("token_blend: unknown dtype %d", dtype);
+  return sprout_check_launch("token_blend");
+}
+
+SPROUT_API int sprout_gated_group_norm(const float* o, const void* gate, int gate_stride, int gate_dtype, const float* weight, int period, void* out,
                                        int dtype, int rows, int width, int groups, float eps, int gate_first, int act,
                                        cudaStream_t stream) {
   SPROUT_REQUIRE(o && (gate || !gate_first) && weight && out && rows > 0 && width > 0 && eps > 0, "gated_group_norm: bad arguments");
   SPROUT_REQUIRE(groups > 0 && groups <= 65535 && width % groups == 0 && period > 0 && (!gate || gate_stride >= width),
                  "gated_group_norm: the row must divide into the groups, gate rows must hold the row");
+  SPROUT_REQUIRE(!gate || gate_dtype == dtype || gate_dtype == SPROUT_F32, "gated_group_norm: the gate is of out's type or float32");
   if (dtype == SPROUT_F32)
-    sprout_launch(gated_group_norm_kernel<float>, dim3(rows, groups), dim3(128), 0, stream, o, (const float*)gate, gate_stride, weight,
+    sprout_launch(gated_group_norm_kernel<float, float>, dim3(rows, groups), dim3(128), 0, stream, o, (const float*)gate, gate_stride, weight,
                   period, (float*)out, width, groups, eps, gate_first, act);
+  else if (dtype == SPROUT_BF16 && gate && gate_dtype == SPROUT_F32)
+    sprout_launch(gated_group_norm_kernel<float, __nv_bfloat16>, dim3(rows, groups), dim3(128), 0, stream, o, (const float*)gate,
+                  gate_stride, weight, period, (__nv_bfloat16*)out, width, groups, eps, gate_first, act);
   else if (dtype == SPROUT_BF16)
-    sprout_launch(gated_group_norm_kernel<__nv_bfloat16>, dim3(rows, groups), dim3(128), 0, stream, o, (const __nv_bfloat16*)gate,
+    sprout_launch(gated_group_norm_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(rows, groups), dim3(128), 0, stream, o, (const __nv_bfloat16*)gate,
                   gate_stride, weight, period, (__nv_bfloat16*)out, width, groups, eps, gate_first, act);
   else
     return sprout_fail("gated_group_norm: unknown dtype %d", dtype);

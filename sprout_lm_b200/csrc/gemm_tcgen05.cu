@@ -18,6 +18,8 @@
 //       is filled by weight rows instead of by a handful of tokens.
 //       With split_k > 1 the K range is divided among CTAs (grid.z) and the partial sums are
 //       added into the float32 output with atomics (residual epilogue only).
+// Groups of output features may read columns of their own of A (several matrices over several inputs in one launch): A is then
+// [M, groups * K], and the features of group g multiply A's columns [g K, (g + 1) K).
 //
 // Every wait on an mbarrier is bounded; a wait that runs out sets SPROUT_STATUS_WAIT_TIMEOUT,
 // the CTA stops issuing, waits (bounded) for its copies in flight, frees its TMEM and returns.
@@ -59,6 +61,7 @@ struct Params {
   int ldo;
   int k_blocks_per_split;
   int* status;
+  int group_rows, groups;  // output features per group of A's columns (a multiple of every tile); groups 1: one A for all
   // weights on M only: the tokens' operand made in the kernel instead of copied: bfloat16(x * gain) of the
   // float32 rows x [M, K] (row stride ldx), written by the epilogue warps into the stages' token tiles
   const float* x32; const float* gain; int ldx;
@@ -201,6 +204,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
 #endif
       }
       int x = k.kb_begin * BLOCK_K;
+      const int act_x = p.groups > 1 ? min((SWAP ? k.row0 : k.col0) / p.group_rows, p.groups - 1) * p.K : 0;
       for (int i = 0; i < k.num_kb; i++, it++, x += BLOCK_K) {
         const uint32_t count_addr = count_base + 8 * s;
         if (i >= early) {
@@ -208,7 +212,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
           if (rank == 0) mbar_expect_tx_addr(full_base + 8 * s, STAGE_TX);
           copy(stage_addr + W_OFF, weight_map, count_addr, x, weight_row);
         }
-        if (!made_here) copy(stage_addr + X_OFF, act_map, count_addr, x, act_row);
+        if (!made_here) copy(stage_addr + X_OFF, act_map, count_addr, act_x + x, act_row);
         issued = it + 1;
         if (++s == L::STAGES) { s = 0; parity ^= 1; stage_addr = smem_base; } else stage_addr += L::STAGE_BYTES;
       }
@@ -549,9 +553,12 @@ int launch(const CUtensorMap& rows_map, const CUtensorMap& cols_map, const CUten
 // atomics.
 // residual == 2: the SwiGLU epilogue (no bias; out is bfloat16 [M, N/2]; N a multiple of 16); residual == 3: the same with
 // the tanh form of gelu on the gate.
+// groups > 1: A is [M, groups * K]; output features [g * group_rows, (g + 1) * group_rows) multiply A's columns [g K, (g + 1) K)
+// (the last group takes the features that are left).  In the last k-block of a K that is no multiple of 64 the next
+// group's columns meet weights that are zero (beyond W's rows): A must be finite.
 SPROUT_API int sprout_gemm_bf16(const void* A, const void* W, const float* bias, void* out, int out_dtype,
                                 int residual, int M, int N, int K, int lda, int ldo, int orientation,
-                                int split_k, int* status, cudaStream_t stream) {
+                                int split_k, int groups, int group_rows, int* status, cudaStream_t stream) {
   const bool swiglu = residual == 2 || residual == 3;
   const int gate_gelu = residual == 3 ? 1 : 0;
   if (swiglu) {
@@ -564,7 +571,10 @@ SPROUT_API int sprout_gemm_bf16(const void* A, const void* W, const float* bias,
   SPROUT_REQUIRE(K % 8 == 0 && lda % 8 == 0, "gemm_bf16: K (%d) and the row stride of A (%d) must be multiples of 8 "
                  "(TMA rows start on 16-byte boundaries)", K, lda);
   SPROUT_REQUIRE(((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0, "gemm_bf16: operands must be 16-byte aligned");
-  SPROUT_REQUIRE(lda >= K && (swiglu || ldo >= N), "gemm_bf16: row strides smaller than the rows");
+  if (groups < 1) groups = 1;
+  SPROUT_REQUIRE(groups == 1 || (group_rows > 0 && group_rows % BLOCK_M == 0 && (long long)group_rows * (groups - 1) < N),
+                 "gemm_bf16: groups of output features must be multiples of %d (got %d)", BLOCK_M, group_rows);
+  SPROUT_REQUIRE(lda >= groups * K && (swiglu || ldo >= N), "gemm_bf16: row strides smaller than the rows");
   SPROUT_REQUIRE(out_dtype == SPROUT_F32 || out_dtype == SPROUT_BF16, "gemm_bf16: unknown output dtype %d", out_dtype);
   SPROUT_REQUIRE(!residual || out_dtype == SPROUT_F32, "gemm_bf16: a residual needs a float32 output");
   // Which operand fills the MMA's 128 rows (orientation 0 picks): the weights for a stream of
@@ -587,6 +597,7 @@ SPROUT_API int sprout_gemm_bf16(const void* A, const void* W, const float* bias,
   p.epilogue = swiglu ? EPI_SWIGLU : residual ? (split_k > 1 ? EPI_RESIDUAL_ATOMIC : EPI_RESIDUAL) : EPI_STORE;
   p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.status = status;
   p.x32 = nullptr; p.gain = nullptr; p.ldx = 0;
+  p.groups = groups; p.group_rows = group_rows;
   const int total_kb = (K + BLOCK_K - 1) / BLOCK_K;
   if (split_k > total_kb) split_k = total_kb;
   p.k_blocks_per_split = (total_kb + split_k - 1) / split_k;
@@ -596,7 +607,7 @@ SPROUT_API int sprout_gemm_bf16(const void* A, const void* W, const float* bias,
   if (swap) {
     const int bn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
     if (tensor_map(W, N, K, K, BLOCK_M, &map_w)) return 1;
-    if (tensor_map(A, M, K, lda, bn, &map_a)) return 1;
+    if (tensor_map(A, M, groups * K, lda, bn, &map_a)) return 1;
     const long long work = (long long)((N + BLOCK_M - 1) / BLOCK_M) * ((M + bn - 1) / bn) * split_k;
     SPROUT_REQUIRE(work <= 0x7fffffffLL, "gemm_bf16: too many tiles");
     switch (bn) {
@@ -618,15 +629,15 @@ SPROUT_API int sprout_gemm_bf16(const void* A, const void* W, const float* bias,
   // 41 -> 39 us, 8192 tokens 145 -> 134 us; on narrower tiles single CTAs are as fast).
   int bn = 128;
   split_k = 1;
-  const bool pair = orientation == 4 || (orientation != 3 && N % 256 == 0 && !(orientation == 0 && swiglu && M <= 128));
+  const bool pair = orientation == 4 || (orientation != 3 && N % 256 == 0 && (groups == 1 || group_rows % 256 == 0) && !(orientation == 0 && swiglu && M <= 128));
   if (pair) {
-    bn = N % 256 == 0 ? 256 : 128;
+    bn = N % 256 == 0 && (groups == 1 || group_rows % 256 == 0) ? 256 : 128;
   } else if (orientation != 3) {
     const int widths[4] = {128, 192, 224, 256};
     const long long row_tiles = (M + BLOCK_M - 1) / BLOCK_M;
     long long best = -1;
     for (int width : widths) {
-      if (width != 128 && N % width != 0) continue;
+      if (width != 128 && (N % width != 0 || (groups > 1 && group_rows % width != 0))) continue;
       for (int split = 1; split <= (reduce ? 4 : 1); split++) {
         const int kb = (total_kb + split - 1) / split;
         if (split > 1 && kb < 4) break;
@@ -639,7 +650,7 @@ SPROUT_API int sprout_gemm_bf16(const void* A, const void* W, const float* bias,
   }
   p.k_blocks_per_split = (total_kb + split_k - 1) / split_k;
   split_k = (total_kb + p.k_blocks_per_split - 1) / p.k_blocks_per_split;
-  if (tensor_map(A, M, K, lda, BLOCK_M, &map_a)) return 1;
+  if (tensor_map(A, M, groups * K, lda, BLOCK_M, &map_a)) return 1;
   if (tensor_map(W, N, K, K, pair ? bn / 2 : bn, &map_w)) return 1;
   const long long work = (long long)((N + bn - 1) / bn) * ((M + (pair ? 2 : 1) * BLOCK_M - 1) / ((pair ? 2 : 1) * BLOCK_M)) * split_k;
   SPROUT_REQUIRE(work <= 0x7fffffffLL, "gemm_bf16: too many tiles");
@@ -678,6 +689,7 @@ SPROUT_API int sprout_gemm_bf16_unscaled(const float* x, int ldx, const float* g
   p.bias = nullptr; p.out = out; p.out_is_f32 = 1; p.epilogue = EPI_RESIDUAL_ATOMIC;
   p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.status = status;
   p.x32 = x; p.gain = gain; p.ldx = ldx;
+  p.groups = 1; p.group_rows = 0;
   const int total_kb = (K + BLOCK_K - 1) / BLOCK_K;
   if (split_k < 1) split_k = 1;
   if (split_k > total_kb) split_k = total_kb;

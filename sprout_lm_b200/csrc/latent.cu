@@ -14,10 +14,10 @@
 //  * headwise_gemm:     out[t, h, :] = W[h] a[t, h, :], one small matrix per head.
 //  * latent_attention_simple: causal attention of (token, head) rows over the latent cache rows,
 //                       all heads reading the same row; the value is the row's first `rank`
-//                       elements; optional sink term in the softmax denominator.
+//                       elements; optional sink term in the softmax denominator, optional sliding window.
 //  * depth_average:     keeps a layer's result in a history and replaces the stream by a weighted
 //                       sum of the history so far.
-//  * softcap:           x = cap * tanh(x / cap), in place.
+//  * softcap:           x = cap * tanh(x / cap), in place, x multiplied by a factor first.
 #include "attention_bf16.cuh"
 
 using namespace sprout_attn;
@@ -411,7 +411,7 @@ latent_attention_simple_kernel(const T* __restrict__ qlat, const T* __restrict__
                                const int* __restrict__ block_table, int table_stride,
                                const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                                const float* __restrict__ sink, T* __restrict__ out, int heads, int width, int rank,
-                               int page_tokens, int num_pages, float scale, int* status) {
+                               int page_tokens, int num_pages, float scale, int window, int* status) {
   extern __shared__ float smem[];
   float* qs = smem;                       // width
   float* probs = qs + width;              // CHUNK
@@ -428,9 +428,10 @@ latent_attention_simple_kernel(const T* __restrict__ qlat, const T* __restrict__
   float acc[MAX_V];
 #pragma unroll
   for (int i = 0; i < MAX_V; i++) acc[i] = 0.f;
-  for (int base = 0; base <= pos; base += CHUNK) {
+  const int lowest = window > 0 ? max(0, pos - window + 1) : 0;         // the first position the query sees
+  for (int base = lowest / CHUNK * CHUNK; base <= pos; base += CHUNK) {
     const int p = base + tid;
-    bool valid = p <= pos;
+    bool valid = p >= lowest && p <= pos;
     long long offset = 0;
     if (valid) {
       const int page = table[p / page_tokens];
@@ -513,11 +514,12 @@ __global__ void depth_average_vec_kernel(float4* __restrict__ history, float4* _
   }
 }
 
-__global__ void softcap_kernel(float* __restrict__ x, float cap, long long count) {
+// x = cap * tanh(factor * x / cap); cap 0: x = factor * x
+__global__ void softcap_kernel(float* __restrict__ x, float cap, float factor, long long count) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < count; i += (long long)gridDim.x * blockDim.x)
-    x[i] = cap * tanhf(x[i] / cap);
+    x[i] = cap > 0.f ? cap * tanhf((factor * x[i]) / cap) : factor * x[i];
 }
 
 inline int flat_grid(long long count, int threads) {
@@ -668,21 +670,22 @@ SPROUT_API int sprout_headwise_gemm(const void* a, long long a_row, long long a_
 SPROUT_API int sprout_latent_attention_simple(const void* qlat, const void* cache, const int* block_table, int table_stride,
                                               const int* seq_of_token, const int* positions, const float* sink, void* out,
                                               int dtype, int tokens, int heads, int width, int rank, int page_tokens,
-                                              int num_pages, float scale, int* status, cudaStream_t stream) {
+                                              int num_pages, float scale, int window, int* status, cudaStream_t stream) {
   SPROUT_REQUIRE(qlat && cache && block_table && seq_of_token && positions && out && status, "latent_attention_simple: null pointer");
   SPROUT_REQUIRE(tokens > 0 && heads > 0 && heads <= 65535 && rank > 0 && width >= rank && page_tokens > 0 && num_pages > 0,
                  "latent_attention_simple: sizes do not fit");
+  SPROUT_REQUIRE(window >= 0, "latent_attention_simple: a window is not negative");
   SPROUT_REQUIRE(rank <= MAX_V * CHUNK, "latent_attention_simple: latent size %d above %d", rank, MAX_V * CHUNK);
   const size_t smem = (size_t)(width + (width & 1) + CHUNK + 34) * sizeof(float) + CHUNK * sizeof(long long);
   dim3 grid(tokens, heads);
   if (dtype == SPROUT_F32)
     sprout_launch(latent_attention_simple_kernel<float>, grid, dim3(CHUNK), smem, stream, (const float*)qlat, (const float*)cache,
                   block_table, table_stride, seq_of_token, positions, sink, (float*)out, heads, width, rank, page_tokens,
-                  num_pages, scale, status);
+                  num_pages, scale, window, status);
   else if (dtype == SPROUT_BF16)
     sprout_launch(latent_attention_simple_kernel<__nv_bfloat16>, grid, dim3(CHUNK), smem, stream, (const __nv_bfloat16*)qlat,
                   (const __nv_bfloat16*)cache, block_table, table_stride, seq_of_token, positions, sink, (__nv_bfloat16*)out,
-                  heads, width, rank, page_tokens, num_pages, scale, status);
+                  heads, width, rank, page_tokens, num_pages, scale, window, status);
   else
     return sprout_fail("latent_attention_simple: unknown dtype %d", dtype);
   return sprout_check_launch("latent_attention_simple");
@@ -698,8 +701,8 @@ SPROUT_API int sprout_depth_average(float* history, float* x, const float* weigh
   return sprout_check_launch("depth_average");
 }
 
-SPROUT_API int sprout_softcap(float* x, float cap, long long count, cudaStream_t stream) {
-  SPROUT_REQUIRE(x && count > 0 && cap > 0.f, "softcap: null pointer, no elements or a cap that is not positive");
-  sprout_launch(softcap_kernel, dim3(flat_grid(count, 256)), dim3(256), 0, stream, x, cap, count);
+SPROUT_API int sprout_softcap(float* x, float cap, float factor, long long count, cudaStream_t stream) {
+  SPROUT_REQUIRE(x && count > 0 && cap >= 0.f, "softcap: null pointer, no elements or a negative cap");
+  sprout_launch(softcap_kernel, dim3(flat_grid(count, 256)), dim3(256), 0, stream, x, cap, factor, count);
   return sprout_check_launch("softcap");
 }

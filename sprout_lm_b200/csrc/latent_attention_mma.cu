@@ -15,6 +15,9 @@
 //    its keys; 4 warps per block of value columns take a quarter of every stage each and are merged
 //    through shared memory; the ranges' partial sums go through float32 scratch to a merge kernel,
 //    which also adds the sink.
+//
+// With a window a row sees its own position and the window - 1 before it: the walk starts at the first key that any of
+// the CTA's rows sees, keys before a row's own first are masked, and split ranges are counted from the token's first key.
 #include "attention_bf16.cuh"
 #include "tcgen05.cuh"
 
@@ -36,6 +39,7 @@ struct LatentParams {
   float* part_o;                  // [requests, splits, heads, rank]   (split keys)
   float* part_ml;                 // [requests, splits, heads, 2]
   int requests, heads, width, rank, page_tokens, num_pages, split_keys, splits;
+  int window;                     // 0: every earlier position
   float scale;
   int* status;
 };
@@ -99,17 +103,17 @@ __device__ __forceinline__ void scores_block(const __nv_bfloat16* sQ, const __nv
 // The same warp, from its scores on: mask, online softmax, O += P V over the warp's value columns.
 template <int DVC, int NT>
 __device__ __forceinline__ void softmax_values_block(float (&s)[NT][4], const __nv_bfloat16* tK, int stride, int col0, int col_end,
-                                                     int key0, int limit0, int limit1, bool mask, float scale_log2, float& m0,
-                                                     float& m1, float& l0, float& l1, float (&o)[DVC / 8][4], int lane) {
+                                                     int key0, int limit0, int limit1, int low0, int low1, bool mask, float scale_log2,
+                                                     float& m0, float& m1, float& l0, float& l1, float (&o)[DVC / 8][4], int lane) {
   const int qc = lane & 3;
   if (mask) {
 #pragma unroll
     for (int i = 0; i < NT; i++) {
       const int key = key0 + i * 8 + qc * 2;
-      if (key > limit0) s[i][0] = -INFINITY;
-      if (key + 1 > limit0) s[i][1] = -INFINITY;
-      if (key > limit1) s[i][2] = -INFINITY;
-      if (key + 1 > limit1) s[i][3] = -INFINITY;
+      if (key > limit0 || key < low0) s[i][0] = -INFINITY;
+      if (key + 1 > limit0 || key + 1 < low0) s[i][1] = -INFINITY;
+      if (key > limit1 || key < low1) s[i][2] = -INFINITY;
+      if (key + 1 > limit1 || key + 1 < low1) s[i][3] = -INFINITY;
     }
   }
   float t0 = -INFINITY, t1 = -INFINITY;
@@ -159,16 +163,6 @@ __device__ __forceinline__ void softmax_values_block(float (&s)[NT][4], const __
   }
 }
 
-template <int DVC, int NT>
-__device__ __forceinline__ void attend_block(const __nv_bfloat16* sQ, const __nv_bfloat16* tK, int stride, int width,
-                                             int col0, int col_end, int key0, int limit0, int limit1, bool mask,
-                                             float scale_log2, float& m0, float& m1, float& l0, float& l1,
-                                             float (&o)[DVC / 8][4], int lane) {
-  float s[NT][4];
-  scores_block<NT>(sQ, tK, stride, 0, width / 16, s, lane);
-  softmax_values_block<DVC, NT>(s, tK, stride, col0, col_end, key0, limit0, limit1, mask, scale_log2, m0, m1, l0, l1, o, lane);
-}
-
 // One stage of key rows: each of the first KEYS threads finds its row's place in the pool and starts one bulk copy
 // of the whole row into shared memory (a row beyond the range is cleared instead); every one of them arrives on the
 // stage's mbarrier (initialised with a count of KEYS), a copying thread together with its row's bytes.
@@ -177,11 +171,12 @@ __device__ __forceinline__ void bulk_row(void* dst, const void* src, uint32_t by
                ::"r"(smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
 }
 // The page of a thread's key row in a stage (read one stage ahead of its use, so that the load's latency is not on the
-// stage's path): -2 for a key beyond the range, else the block table's entry.
+// stage's path): -2 for a key before `lowest` or beyond the range (its page may have been given back), else the block
+// table's entry.
 template <int KEYS>
-__device__ __forceinline__ int page_ahead(const LatentParams& p, const int* table, int first_key, int last_key, int tid) {
+__device__ __forceinline__ int page_ahead(const LatentParams& p, const int* table, int first_key, int lowest, int last_key, int tid) {
   const int key = first_key + tid;
-  return (tid < KEYS && key <= last_key) ? table[key / p.page_tokens] : -2;
+  return (tid < KEYS && key >= lowest && key <= last_key) ? table[key / p.page_tokens] : -2;
 }
 template <int KEYS>
 __device__ __forceinline__ void issue_stage(const LatentParams& p, int page, int first_key, __nv_bfloat16* dst, int stride,
@@ -275,20 +270,23 @@ latent_attention_rows_kernel(const LatentParams p) {
   __syncthreads();
   const int last_row = min(rows_total, row_base + ROWS) - 1 - row_base;
   const int max_limit = s_limit[last_row];
-  const int stages = max_limit / KEYS + 1;
+  // rows are in the tokens' order: the first row's window reaches furthest back
+  const int lowest = p.window > 0 ? max(0, s_limit[0] - p.window + 1) : 0;
+  const int first_stage = lowest / KEYS, stages = max_limit / KEYS + 1;
   for_pieces(ROWS, p.width / 8, tid, THREADS, [&](int row, int c) {
     __nv_bfloat16* dst = sQ + row * stride + c * 8;
     if (s_token[row] >= 0) cp_async16(dst, p.q + ((size_t)s_token[row] * p.heads + s_head[row]) * p.width + c * 8);
     else *(uint4*)dst = make_uint4(0, 0, 0, 0);
   });
   cp_async_commit();
-  issue_stage<KEYS>(p, page_ahead<KEYS>(p, table, 0, max_limit, tid), 0, sK, stride, &s_bar[0], tid);
-  int page_next = page_ahead<KEYS>(p, table, KEYS, max_limit, tid);       // of the stage after: read now, used at the loop's next turn
+  issue_stage<KEYS>(p, page_ahead<KEYS>(p, table, first_stage * KEYS, lowest, max_limit, tid), first_stage * KEYS, sK, stride, &s_bar[0], tid);
+  int page_next = page_ahead<KEYS>(p, table, (first_stage + 1) * KEYS, lowest, max_limit, tid);       // of the stage after: read now, used at the loop's next turn
   cp_async_wait<0>();                                 // this thread's pieces of the query rows; the loop's first barrier publishes them
 
   const int gr = lane >> 2, qc = lane & 3;
   const int my_row0 = group * 16 + gr, my_row1 = my_row0 + 8;
   const int limit0 = s_limit[my_row0], limit1 = s_limit[my_row1];
+  const int low0 = p.window > 0 ? limit0 - p.window + 1 : 0, low1 = p.window > 0 ? limit1 - p.window + 1 : 0;
   const float scale_log2 = p.scale * 1.4426950408889634f;
   // a sink starts the running maximum (in units of the unscaled score) and counts once in the sum
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
@@ -301,20 +299,21 @@ latent_attention_rows_kernel(const LatentParams p) {
   for (int i = 0; i < DVC / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   const int warp_min_limit = s_limit[min(group * 16, last_row)];
   const int warp_limit = s_limit[min(group * 16 + 15, last_row)];
+  const int warp_low = p.window > 0 ? warp_min_limit - p.window + 1 : 0, warp_high = p.window > 0 ? warp_limit - p.window + 1 : 0;
   const bool active = group * 16 <= last_row && col0 < p.rank;
   const bool paired = CHUNKS == 2 && (blockIdx.y * CHUNKS + 1) * DVC < p.rank;      // both blocks of value columns exist
 
-  for (int t = 0; t < stages; t++) {
-    const int buf = t & 1;
+  for (int t = first_stage; t < stages; t++) {
+    const int buf = (t - first_stage) & 1;
     __syncthreads();                                  // every warp is done with the other buffer; cleared rows are visible
     if (s_failed) break;
     if (t + 1 < stages) {
       issue_stage<KEYS>(p, page_next, (t + 1) * KEYS, sK + (buf ^ 1) * KEYS * stride, stride, &s_bar[buf ^ 1], tid);
-      page_next = page_ahead<KEYS>(p, table, (t + 2) * KEYS, max_limit, tid);
+      page_next = page_ahead<KEYS>(p, table, (t + 2) * KEYS, lowest, max_limit, tid);
     }
-    stage_landed(&s_bar[buf], (t >> 1) & 1, p.status, &s_failed);
+    stage_landed(&s_bar[buf], ((t - first_stage) >> 1) & 1, p.status, &s_failed);
     const int key0 = t * KEYS;
-    if (active && key0 <= warp_limit) {
+    if (active && key0 <= warp_limit && key0 + KEYS > warp_low) {
       constexpr int NT = KEYS / 8;
       const __nv_bfloat16* tK = sK + buf * KEYS * stride;
       float sc[NT][4];
@@ -336,8 +335,8 @@ latent_attention_rows_kernel(const LatentParams p) {
       } else {
         scores_block<NT>(sQ + group * 16 * stride, tK, stride, 0, p.width / 16, sc, lane);
       }
-      softmax_values_block<DVC, NT>(sc, tK, stride, col0, col_end, key0, limit0, limit1, key0 + KEYS - 1 > warp_min_limit,
-                                    scale_log2, m0, m1, l0, l1, o, lane);
+      softmax_values_block<DVC, NT>(sc, tK, stride, col0, col_end, key0, limit0, limit1, low0, low1,
+                                    key0 + KEYS - 1 > warp_min_limit || key0 < warp_high, scale_log2, m0, m1, l0, l1, o, lane);
     }
   }
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
@@ -387,8 +386,9 @@ latent_attention_split_kernel(const LatentParams p) {
   const int col0 = cta_col0 + chunk * DVC, col_end = min(p.rank, col0 + DVC);
   const int split = blockIdx.z;
   const int limit = p.context_lens[r] - 1;            // the token's own position: the last key it sees
+  const int lowest = p.window > 0 ? max(0, limit - p.window + 1) : 0;
   // the last range runs to the token's position, however the ranges were planned
-  const int first = split * p.split_keys, last = split == p.splits - 1 ? limit : min(limit, first + p.split_keys - 1);
+  const int first = lowest + split * p.split_keys, last = split == p.splits - 1 ? limit : min(limit, first + p.split_keys - 1);
   const int stages = last >= first ? (last - first) / KEYS + 1 : 0;
   const int* table = p.block_table + (size_t)r * p.table_stride;
   const int token = p.q_start[r];
@@ -400,9 +400,9 @@ latent_attention_split_kernel(const LatentParams p) {
   cp_async_commit();
   __syncthreads();                                    // the mbarriers are initialised
   for (int t = 0; t < NSTAGES - 1 && t < stages; t++)
-    issue_stage<KEYS>(p, page_ahead<KEYS>(p, table, first + t * KEYS, last, tid), first + t * KEYS, sK + t * KEYS * stride, stride,
+    issue_stage<KEYS>(p, page_ahead<KEYS>(p, table, first + t * KEYS, first, last, tid), first + t * KEYS, sK + t * KEYS * stride, stride,
                       &s_bar[t], tid);
-  int page_next = page_ahead<KEYS>(p, table, first + (NSTAGES - 1) * KEYS, last, tid);   // read now, used at the loop's next turn
+  int page_next = page_ahead<KEYS>(p, table, first + (NSTAGES - 1) * KEYS, first, last, tid);   // read now, used at the loop's next turn
   cp_async_wait<0>();
 
   const int gr = lane >> 2, qc = lane & 3;
@@ -420,7 +420,7 @@ latent_attention_split_kernel(const LatentParams p) {
     if (t + NSTAGES - 1 < stages) {
       const int ahead = (t + NSTAGES - 1) % NSTAGES;  // the buffer that was worked on last
       issue_stage<KEYS>(p, page_next, first + (t + NSTAGES - 1) * KEYS, sK + ahead * KEYS * stride, stride, &s_bar[ahead], tid);
-      page_next = page_ahead<KEYS>(p, table, first + (t + NSTAGES) * KEYS, last, tid);
+      page_next = page_ahead<KEYS>(p, table, first + (t + NSTAGES) * KEYS, first, last, tid);
     }
     stage_landed(&s_bar[buf], (t / NSTAGES) & 1, p.status, &s_failed);
     const int key0 = first + t * KEYS + quarter * 16; // this warp's share of the stage
@@ -449,8 +449,8 @@ latent_attention_split_kernel(const LatentParams p) {
       } else {
         scores_block<2>(sQ, tK, stride, 0, steps, sc, lane);
       }
-      softmax_values_block<DVC, 2>(sc, tK, stride, col0, col_end, key0, last, last, key0 + 15 > last, scale_log2, m0, m1, l0, l1,
-                                   o, lane);
+      softmax_values_block<DVC, 2>(sc, tK, stride, col0, col_end, key0, last, last, 0, 0, key0 + 15 > last, scale_log2, m0, m1,
+                                   l0, l1, o, lane);
     }
   }
   __syncthreads();                                    // every warp is done with the stages: they become the exchange area
@@ -574,7 +574,8 @@ SPROUT_API int sprout_latent_attention_mma(const void* q, const void* cache, con
                                            const int* q_start, const int* positions, const int* context_lens,
                                            const float* sink, void* out, float* scratch, int tokens, int requests,
                                            int heads, int width, int rank, int page_tokens, int num_pages, int splits,
-                                           int split_keys, float scale, int* status, cudaStream_t stream) {
+                                           int split_keys, float scale, int window, int* status, cudaStream_t stream) {
+  SPROUT_REQUIRE(window >= 0, "latent_attention_mma: a window is not negative");
   SPROUT_REQUIRE(q && cache && block_table && q_start && positions && out && status, "latent_attention_mma: null pointer");
   SPROUT_REQUIRE(tokens > 0 && requests > 0 && heads > 0 && page_tokens > 0 && num_pages > 0 && scale > 0.f,
                  "latent_attention_mma: sizes and scale must be positive");
@@ -584,7 +585,7 @@ SPROUT_API int sprout_latent_attention_mma(const void* q, const void* cache, con
   p.q = (const __nv_bfloat16*)q; p.cache = (const __nv_bfloat16*)cache; p.block_table = block_table; p.table_stride = table_stride;
   p.q_start = q_start; p.positions = positions; p.context_lens = context_lens; p.sink = sink; p.out = (__nv_bfloat16*)out;
   p.requests = requests; p.heads = heads; p.width = width; p.rank = rank; p.page_tokens = page_tokens; p.num_pages = num_pages;
-  p.split_keys = split_keys; p.splits = splits; p.scale = scale; p.status = status;
+  p.split_keys = split_keys; p.splits = splits; p.scale = scale; p.window = window; p.status = status;
   p.part_o = scratch; p.part_ml = scratch ? scratch + (size_t)requests * splits * heads * rank : nullptr;
   const Division d = divide(rank);
   const size_t row_bytes = (size_t)(width + 8) * 2;

@@ -3,7 +3,8 @@
 //                    rows may be selected by index.
 //  * norm_add:       x += layernorm(y) * w_b, and, when asked, h = layernorm(x) * w_next of the new x:
 //                    the norm after a sublayer, the residual sum and the norm before the next
-//                    sublayer in one launch.
+//                    sublayer in one launch.  Both norms may be RMS norms instead (nothing is subtracted:
+//                    mean = 0), and y may be cleared behind the read, ready for the next sublayer's sums.
 //  * gated_rmsnorm:  out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate).
 //  * relu2, glu_clamped: activations between the two products of a feed-forward.
 // One block per row, or (rows of 128 to 4,096 elements in steps the kernels are built for) a warp per row with the row
@@ -15,11 +16,16 @@ namespace {
 
 constexpr int THREADS = 256;
 
-// mean and 1 / sqrt(var + eps) of a row held in shared memory (two passes: the deviations are exact)
-__device__ __forceinline__ void row_moments(const float* row, int width, float eps, float* scratch, float& mean, float& rstd) {
-  float s = 0.f;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) s += row[i];
-  mean = block_sum(s, scratch) / (float)width;
+// mean and 1 / sqrt(var + eps) of a row held in shared memory (two passes: the deviations are exact); `centered` 0: the
+// mean is taken as 0, which makes it the root mean square
+__device__ __forceinline__ void row_moments(const float* row, int width, float eps, int centered, float* scratch, float& mean,
+                                            float& rstd) {
+  mean = 0.f;
+  if (centered) {
+    float s = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) s += row[i];
+    mean = block_sum(s, scratch) / (float)width;
+  }
   float q = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) {
     const float d = row[i] - mean;
@@ -41,25 +47,28 @@ layernorm_kernel(const float* __restrict__ x, const float* __restrict__ gain, co
   for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = x[src + i];
   __syncthreads();
   float mean, rstd;
-  row_moments(row, width, eps, scratch, mean, rstd);
+  row_moments(row, width, eps, 1, scratch, mean, rstd);
   TO* dst = out + (size_t)blockIdx.x * width;
   for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_float<TO>((row[i] - mean) * rstd * gain[i] + (bias ? bias[i] : 0.f));
 }
 
 template <typename TO>
 __global__ void __launch_bounds__(THREADS)
-norm_add_kernel(const float* __restrict__ y, const float* __restrict__ gain, float* __restrict__ x,
-                const float* __restrict__ next_gain, TO* __restrict__ h, int width, float eps) {
+norm_add_kernel(float* __restrict__ y, const float* __restrict__ gain, float* __restrict__ x,
+                const float* __restrict__ next_gain, TO* __restrict__ h, int width, float eps, int centered, int clear) {
   extern __shared__ float smem[];
   float* row = smem;
   float* scratch = smem + width;
   pdl_launch_dependents();
   pdl_wait();
   const size_t at = (size_t)blockIdx.x * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) row[i] = y[at + i];
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    row[i] = y[at + i];
+    if (clear) y[at + i] = 0.f;
+  }
   __syncthreads();
   float mean, rstd;
-  row_moments(row, width, eps, scratch, mean, rstd);
+  row_moments(row, width, eps, centered, scratch, mean, rstd);
   for (int i = threadIdx.x; i < width; i += blockDim.x) {      // each thread rewrites the elements it read
     const float v = x[at + i] + (row[i] - mean) * rstd * gain[i];
     x[at + i] = v;
@@ -67,7 +76,7 @@ norm_add_kernel(const float* __restrict__ y, const float* __restrict__ gain, flo
   }
   if (next_gain == nullptr) return;
   __syncthreads();
-  row_moments(row, width, eps, scratch, mean, rstd);
+  row_moments(row, width, eps, centered, scratch, mean, rstd);
   for (int i = threadIdx.x; i < width; i += blockDim.x) h[at + i] = from_float<TO>((row[i] - mean) * rstd * next_gain[i]);
 }
 
@@ -83,11 +92,14 @@ __device__ __forceinline__ void store_four(TO* dst, float a, float b, float c, f
 }
 
 template <int NV>
-__device__ __forceinline__ void warp_moments(const float4 (&v)[NV], float eps, float& mean, float& rstd) {
-  float s = 0.f;
+__device__ __forceinline__ void warp_moments(const float4 (&v)[NV], float eps, int centered, float& mean, float& rstd) {
+  mean = 0.f;
+  if (centered) {
+    float s = 0.f;
 #pragma unroll
-  for (int i = 0; i < NV; i++) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
-  mean = warp_sum(s) / (float)(NV * 128);
+    for (int i = 0; i < NV; i++) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    mean = warp_sum(s) / (float)(NV * 128);
+  }
   float q = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; i++) {
@@ -110,7 +122,7 @@ layernorm_rows_kernel(const float* __restrict__ x, const float* __restrict__ gai
 #pragma unroll
   for (int i = 0; i < NV; i++) v[i] = src[i * 32 + lane];
   float mean, rstd;
-  warp_moments<NV>(v, eps, mean, rstd);
+  warp_moments<NV>(v, eps, 1, mean, rstd);
   TO* dst = out + (size_t)row * (NV * 128);
 #pragma unroll
   for (int i = 0; i < NV; i++) {
@@ -123,8 +135,8 @@ layernorm_rows_kernel(const float* __restrict__ x, const float* __restrict__ gai
 
 template <typename TO, int NV>
 __global__ void __launch_bounds__(128)
-norm_add_rows_kernel(const float* __restrict__ y, const float* __restrict__ gain, float* __restrict__ x,
-                     const float* __restrict__ next_gain, TO* __restrict__ h, int count, float eps) {
+norm_add_rows_kernel(float* __restrict__ y, const float* __restrict__ gain, float* __restrict__ x,
+                     const float* __restrict__ next_gain, TO* __restrict__ h, int count, float eps, int centered, int clear) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, row = blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -133,8 +145,12 @@ norm_add_rows_kernel(const float* __restrict__ y, const float* __restrict__ gain
   float4 v[NV];
 #pragma unroll
   for (int i = 0; i < NV; i++) v[i] = ((const float4*)(y + at))[i * 32 + lane];
+  if (clear) {
+#pragma unroll
+    for (int i = 0; i < NV; i++) ((float4*)(y + at))[i * 32 + lane] = make_float4(0.f, 0.f, 0.f, 0.f);
+  }
   float mean, rstd;
-  warp_moments<NV>(v, eps, mean, rstd);
+  warp_moments<NV>(v, eps, centered, mean, rstd);
   float4* stream = (float4*)(x + at);
 #pragma unroll
   for (int i = 0; i < NV; i++) {
@@ -148,7 +164,7 @@ norm_add_rows_kernel(const float* __restrict__ y, const float* __restrict__ gain
     v[i] = s;
   }
   if (next_gain == nullptr) return;
-  warp_moments<NV>(v, eps, mean, rstd);
+  warp_moments<NV>(v, eps, centered, mean, rstd);
 #pragma unroll
   for (int i = 0; i < NV; i++) {
     const float4 g = ((const float4*)next_gain)[i * 32 + lane];
@@ -271,9 +287,10 @@ SPROUT_API int sprout_layernorm(const float* x, const float* gain, const float* 
   return sprout_check_launch("layernorm");
 }
 
-// x [count, width] += layernorm(y) * gain; with next_gain also h = layernorm(x) * next_gain (h in h_dtype).
-SPROUT_API int sprout_norm_add(const float* y, const float* gain, float* x, const float* next_gain, void* h, int h_dtype,
-                               int count, int width, float eps, cudaStream_t stream) {
+// x [count, width] += norm(y) * gain; with next_gain also h = norm(x) * next_gain (h in h_dtype).  The norms are layer norms,
+// or RMS norms when `centered` is 0; `clear` != 0 leaves y zeroed.
+SPROUT_API int sprout_norm_add(float* y, const float* gain, float* x, const float* next_gain, void* h, int h_dtype,
+                               int count, int width, float eps, int centered, int clear, cudaStream_t stream) {
   SPROUT_REQUIRE(y && gain && x && count > 0 && width > 0 && eps > 0, "norm_add: bad arguments");
   SPROUT_REQUIRE((next_gain == nullptr) == (h == nullptr), "norm_add: the next norm's gain and its output go together");
   SPROUT_REQUIRE(width <= 40000, "norm_add: rows of up to 40000 elements (got %d)", width);
@@ -282,8 +299,8 @@ SPROUT_API int sprout_norm_add(const float* y, const float* gain, float* x, cons
       (((uintptr_t)y | (uintptr_t)gain | (uintptr_t)x | (uintptr_t)next_gain | (uintptr_t)h) & 15) == 0) {
     const dim3 grid((count + 3) / 4);
 #define CALL(N)                                                                                                                   \
-    if (h_dtype == SPROUT_F32) sprout_launch(norm_add_rows_kernel<float, N>, grid, dim3(128), 0, stream, y, gain, x, next_gain, (float*)h, count, eps); \
-    else sprout_launch(norm_add_rows_kernel<__nv_bfloat16, N>, grid, dim3(128), 0, stream, y, gain, x, next_gain, (__nv_bfloat16*)h, count, eps);
+    if (h_dtype == SPROUT_F32) sprout_launch(norm_add_rows_kernel<float, N>, grid, dim3(128), 0, stream, y, gain, x, next_gain, (float*)h, count, eps, centered, clear); \
+    else sprout_launch(norm_add_rows_kernel<__nv_bfloat16, N>, grid, dim3(128), 0, stream, y, gain, x, next_gain, (__nv_bfloat16*)h, count, eps, centered, clear);
     SPROUT_FOR_NV(nv, CALL)
 #undef CALL
     return sprout_check_launch("norm_add_rows");
@@ -291,10 +308,10 @@ SPROUT_API int sprout_norm_add(const float* y, const float* gain, float* x, cons
   const size_t smem = (size_t)(width + 34) * sizeof(float);
   if (h_dtype == SPROUT_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    sprout_launch(norm_add_kernel<float>, dim3(count), dim3(THREADS), smem, stream, y, gain, x, next_gain, (float*)h, width, eps);
+    sprout_launch(norm_add_kernel<float>, dim3(count), dim3(THREADS), smem, stream, y, gain, x, next_gain, (float*)h, width, eps, centered, clear);
   } else if (h_dtype == SPROUT_BF16) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(norm_add_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    sprout_launch(norm_add_kernel<__nv_bfloat16>, dim3(count), dim3(THREADS), smem, stream, y, gain, x, next_gain, (__nv_bfloat16*)h, width, eps);
+    sprout_launch(norm_add_kernel<__nv_bfloat16>, dim3(count), dim3(THREADS), smem, stream, y, gain, x, next_gain, (__nv_bfloat16*)h, width, eps, centered, clear);
   } else {
     return sprout_fail("norm_add: unknown dtype %d", h_dtype);
   }

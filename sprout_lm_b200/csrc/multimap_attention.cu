@@ -13,7 +13,8 @@
 //                               the rotation it can divide every vector (or all queries of the token at once, and all
 //                               keys) by its root mean square and multiply it by a weight (one for queries, one for
 //                               keys).  Pairs are (i, i + half) or (2i, 2i + 1).  With tables for the values it also
-//                               turns every value row by its position before it is cached.
+//                               turns every value row by its position before it is cached.  Queries may grow with their
+//                               position p: times 1 + coef * ln(floor((p + 1) / every) + 1).
 // Options of both attention kernels: a mask (a window, a window that also keeps the first positions, chunks), a cap on
 // the scaled scores (cap * tanh(score / cap)), a sink per head in the softmax denominator, a gate per head or per element
 // of the output, and for values that were turned by their position a turn of every head's output back by the query's.
@@ -51,7 +52,7 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
                         int rot, int vdim, int page_tokens, int num_pages, int write, float unit_eps, int value_from_key,
                         const float* __restrict__ q_weight, const float* __restrict__ k_weight, float weight_eps,
                         int weight_whole, int interleaved, const float* __restrict__ v_cos, const float* __restrict__ v_sin,
-                        int* status) {
+                        float growth_coef, int growth_every, int* status) {
   __shared__ float norm_scratch[33];
   pdl_launch_dependents();
   pdl_wait();
@@ -72,6 +73,7 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
     }
   }
   const int kw = maps * dim;
+  const float growth = growth_every > 0 ? 1.0f + growth_coef * logf((float)((pos + 1) / growth_every + 1)) : 1.0f;
   const int vectors = q_vectors + (write ? kv_heads * maps : 0);
   // a norm over the whole projection: one factor for all query vectors of the token, one for all its key vectors
   float whole_q = 1.0f, whole_k = 1.0f;
@@ -93,7 +95,7 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
     if (is_key && page < 0) continue;
     const float* weight = is_key ? k_weight : q_weight;           // the norm before the rotation, when the vector has one
     if (weight_whole && weight != nullptr) weight += (size_t)(is_key ? vec - q_vectors : vec) * dim;
-    if (!is_key && !turn && unit_eps <= 0.f && weight == nullptr) continue;   // nothing to do to this query vector
+    if (!is_key && !turn && unit_eps <= 0.f && weight == nullptr && growth_every <= 0) continue;   // nothing to do to this query vector
     T* src = row + (size_t)vec * dim;                             // the key vectors follow the query vectors
     float vals[ROPE_MAX_PER_LANE], raw[ROPE_MAX_PER_LANE];
     float before = is_key ? whole_k : whole_q;
@@ -131,6 +133,7 @@ rope_maps_append_kernel(T* __restrict__ rows, int row_stride, const int* __restr
     if (unit_eps > 0.f) factor = 1.0f / sqrtf(warp_sum(squares) / (float)dim + unit_eps);
     __syncwarp();                                                 // every partner element was read before any is rewritten
     if (!is_key) {
+      factor *= growth;
 #pragma unroll
       for (int j = 0; j < ROPE_MAX_PER_LANE; j++)
         if (lane + 32 * j < dim) src[lane + 32 * j] = from_float<T>(vals[j] * factor);
@@ -921,8 +924,10 @@ SPROUT_API int sprout_rope_maps_append(void* rows, int row_stride, int dtype, co
                                        int q_vectors, int kv_heads, int maps, int dim, int rot, int vdim, int page_tokens,
                                        int num_pages, int write, float unit_eps, int value_from_key, const float* q_weight,
                                        const float* k_weight, float weight_eps, int weight_whole, int interleaved,
-                                       const float* v_cos, const float* v_sin, int* status, cudaStream_t stream) {
+                                       const float* v_cos, const float* v_sin, float growth_coef, int growth_every, int* status,
+                                       cudaStream_t stream) {
   SPROUT_REQUIRE(rows && positions && status && tokens > 0 && q_vectors > 0 && dim > 0 && maps > 0, "rope_maps_append: bad arguments");
+  SPROUT_REQUIRE(growth_every >= 0, "rope_maps_append: the queries' growth counts positions in positive steps");
   SPROUT_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= dim, "rope_maps_append: the rotated width must be even and at most dim");
   SPROUT_REQUIRE(rot == 0 || (cos_table && sin_table && max_positions > 0), "rope_maps_append: tables are missing");
   SPROUT_REQUIRE(!write || (k_cache && v_cache && seq_of_token && block_table && kv_heads > 0 && vdim > 0 && page_tokens > 0 &&
@@ -937,12 +942,12 @@ SPROUT_API int sprout_rope_maps_append(void* rows, int row_stride, int dtype, co
     sprout_launch(rope_maps_append_kernel<float>, dim3(tokens), dim3(128), 0, stream, (float*)rows, row_stride, positions,
                   seq_of_token, block_table, table_stride, cos_table, sin_table, max_positions, (float*)k_cache,
                   (float*)v_cache, q_vectors, kv_heads, maps, dim, rot, vdim, page_tokens, num_pages, write, unit_eps,
-                  value_from_key, q_weight, k_weight, weight_eps, weight_whole, interleaved, v_cos, v_sin, status);
+                  value_from_key, q_weight, k_weight, weight_eps, weight_whole, interleaved, v_cos, v_sin, growth_coef, growth_every, status);
   else if (dtype == SPROUT_BF16)
     sprout_launch(rope_maps_append_kernel<__nv_bfloat16>, dim3(tokens), dim3(128), 0, stream, (__nv_bfloat16*)rows, row_stride,
                   positions, seq_of_token, block_table, table_stride, cos_table, sin_table, max_positions,
                   (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, q_vectors, kv_heads, maps, dim, rot, vdim, page_tokens,
-                  num_pages, write, unit_eps, value_from_key, q_weight, k_weight, weight_eps, weight_whole, interleaved, v_cos, v_sin, status);
+                  num_pages, write, unit_eps, value_from_key, q_weight, k_weight, weight_eps, weight_whole, interleaved, v_cos, v_sin, growth_coef, growth_every, status);
   else
     return sprout_fail("rope_maps_append: unknown dtype %d", dtype);
   return sprout_check_launch("rope_maps_append");

@@ -2,7 +2,8 @@
 // type of activations (float or bfloat16) is a template parameter.
 //
 //  * unit_act:       out = act(gate) * up for rows laid out [gate: ff | up: ff], or out = act(in) for rows of ff elements;
-//                    act = silu, the tanh form of gelu, or the exact (erf) gelu.  Optionally every row is also multiplied
+//                    act = silu, the tanh form of gelu, the exact (erf) gelu, or tanh.  Rows in may be float32 beside
+//                    bfloat16 rows out.  Optionally every row is also multiplied
 //                    by sigmoid(logit[row]): a gate per token on a sublayer whose last step is linear.
 //  * side_input_few: the whole per-layer token input for a handful of tokens in two launches (see side_gate, rms_add).
 //  * side_gate:      out[t, j] = gelu_tanh(z[t, j]) * table[token[t], first + j]: a per-token row of a table gated by a
@@ -17,24 +18,25 @@
 
 namespace {
 
-enum Activation : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2 };
+enum Activation : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_GELU_ERF = 2, ACT_TANH = 3 };
 
 __device__ __forceinline__ float activate(float z, int act) {
   if (act == ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   if (act == ACT_GELU_ERF) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+  if (act == ACT_TANH) return tanhf(z);
   return z / (1.0f + expf(-z));
 }
 
-template <typename T>
+template <typename TI, typename T>
 __global__ void __launch_bounds__(256)
-unit_act_kernel(const T* __restrict__ in, int in_stride, T* __restrict__ out, int out_stride, long long count, int ff, int act,
+unit_act_kernel(const TI* __restrict__ in, int in_stride, T* __restrict__ out, int out_stride, long long count, int ff, int act,
                 int gated, const float* __restrict__ row_logits, int logit_stride) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long e = blockIdx.x * (long long)blockDim.x + threadIdx.x; e < count; e += (long long)gridDim.x * blockDim.x) {
     const long long r = e / ff;
     const int j = (int)(e - r * ff);
-    const T* row = in + (size_t)r * in_stride;
+    const TI* row = in + (size_t)r * in_stride;
     float v = activate(to_float(row[j]), act);
     if (gated) v *= to_float(row[ff + j]);
     if (row_logits) v *= 1.0f / (1.0f + expf(-row_logits[(size_t)r * logit_stride]));
@@ -275,22 +277,25 @@ SPROUT_API int sprout_side_input_few(float* x, const void* w_gate, const void* w
   return sprout_check_launch("side_input_few (projection)");
 }
 
-SPROUT_API int sprout_unit_act(const void* in, int in_stride, void* out, int out_stride, int dtype, int rows, int ff, int act,
+SPROUT_API int sprout_unit_act(const void* in, int in_stride, int in_dtype, void* out, int out_stride, int dtype, int rows, int ff, int act,
                                int gated, const float* row_logits, int logit_stride, cudaStream_t stream) {
   SPROUT_REQUIRE(in && out && rows > 0 && ff > 0 && in_stride >= (gated ? 2 : 1) * ff && out_stride >= ff, "unit_act: bad arguments");
-  SPROUT_REQUIRE(act >= ACT_SILU && act <= ACT_GELU_ERF, "unit_act: unknown activation %d", act);
+  SPROUT_REQUIRE(act >= ACT_SILU && act <= ACT_TANH, "unit_act: unknown activation %d", act);
   const long long count = (long long)rows * ff;
-  if (dtype == SPROUT_F32)
-    sprout_launch(unit_act_kernel<float>, dim3(blocks_for(count)), dim3(256), 0, stream, (const float*)in, in_stride, (float*)out,
+  if (dtype == SPROUT_F32 && in_dtype == SPROUT_F32)
+    sprout_launch(unit_act_kernel<float, float>, dim3(blocks_for(count)), dim3(256), 0, stream, (const float*)in, in_stride, (float*)out,
                   out_stride, count, ff, act, gated, row_logits, logit_stride);
-  else if (dtype == SPROUT_BF16 && ff % 8 == 0 && in_stride % 8 == 0 && out_stride % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0)
+  else if (dtype == SPROUT_BF16 && in_dtype == SPROUT_F32)
+    sprout_launch(unit_act_kernel<float, __nv_bfloat16>, dim3(blocks_for(count)), dim3(256), 0, stream, (const float*)in, in_stride,
+                  (__nv_bfloat16*)out, out_stride, count, ff, act, gated, row_logits, logit_stride);
+  else if (dtype == SPROUT_BF16 && in_dtype == SPROUT_BF16 && ff % 8 == 0 && in_stride % 8 == 0 && out_stride % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0)
     sprout_launch(unit_act_vec_kernel, dim3(blocks_for(count / 8)), dim3(256), 0, stream, (const __nv_bfloat16*)in, in_stride,
                   (__nv_bfloat16*)out, out_stride, count / 8, ff, act, gated, row_logits, logit_stride);
-  else if (dtype == SPROUT_BF16)
-    sprout_launch(unit_act_kernel<__nv_bfloat16>, dim3(blocks_for(count)), dim3(256), 0, stream, (const __nv_bfloat16*)in, in_stride,
+  else if (dtype == SPROUT_BF16 && in_dtype == SPROUT_BF16)
+    sprout_launch(unit_act_kernel<__nv_bfloat16, __nv_bfloat16>, dim3(blocks_for(count)), dim3(256), 0, stream, (const __nv_bfloat16*)in, in_stride,
                   (__nv_bfloat16*)out, out_stride, count, ff, act, gated, row_logits, logit_stride);
   else
-    return sprout_fail("unit_act: unknown dtype %d", dtype);
+    return sprout_fail("unit_act: unknown dtypes %d, %d", in_dtype, dtype);
   return sprout_check_launch("unit_act");
 }
 

@@ -45,7 +45,7 @@ _SIGNATURES = {
     "sprout_attention_decode_resident_cap": [_I, _I, _I, _I],
     "sprout_attention_prefill": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, ctypes.c_longlong, _P, _P, _P],
     "sprout_attention_prefill_tc_supported": [_I, _I, _I],
-    "sprout_gemm_bf16": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
+    "sprout_gemm_bf16": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "sprout_gemm_bf16_unscaled": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "sprout_ffn_decode": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _P],
     "sprout_ffn_decode_supported": [_I, _I, _I],
@@ -58,17 +58,17 @@ _SIGNATURES = {
     "sprout_latent_kv_append": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P],
     "sprout_latent_query_tail": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "sprout_headwise_gemm": [_P, _L, _L, _P, _P, _L, _L, _I, _I, _I, _I, _I, _P],
-    "sprout_latent_attention_simple": [_P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P],
-    "sprout_latent_attention_mma": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P],
+    "sprout_latent_attention_simple": [_P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
+    "sprout_latent_attention_mma": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
     "sprout_latent_attention_mma_supported": [_I, _I],
     "sprout_depth_average": [_P, _P, _P, _I, _L, _P],
-    "sprout_softcap": [_P, _F, _L, _P],
+    "sprout_softcap": [_P, _F, _F, _L, _P],
     "sprout_layernorm": [_P, _P, _P, _P, _I, _P, _I, _I, _F, _P],
-    "sprout_norm_add": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _P],
+    "sprout_norm_add": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _I, _P],
     "sprout_gated_rmsnorm": [_P, _P, _P, _I, _P, _I, _I, _I, _F, _P],
     "sprout_relu2": [_P, _P, _I, _L, _P],
     "sprout_glu_clamped": [_P, _P, _I, _I, _I, _F, _F, _P],
-    "sprout_rope_maps_append": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _F, _I, _I, _P, _P, _P, _P],
+    "sprout_rope_maps_append": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _F, _I, _I, _P, _P, _F, _I, _P, _P],
     "sprout_multimap_attention_simple": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _I, _P, _P, _I, _I, _F,
                                          _I, _P, _P, _I, _I, _P, _P],
     "sprout_multimap_attention_mma": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _P, _I, _I, _P, _P, _I, _I, _F,
@@ -77,16 +77,17 @@ _SIGNATURES = {
     "sprout_decay_chunks": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "sprout_decay_chunks_supported": [_I, _I, _I],
     "sprout_decay_scan": [_P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P, _P],
-    "sprout_gated_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _P, _P, _P, _F, _F, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P,
+    "sprout_gated_scan": [_P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _P, _P, _P, _P, _F, _F, _I, _I, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P,
                           _I, _I, _I, _P, _P, _P, _P, _I, _I, _I, _P],
     "sprout_delta_rule": [_P, _P, _P, _I, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _P, _P, _I, _P, _I, _P, _P, _P],
     "sprout_causal_conv": [_P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
-    "sprout_gated_group_norm": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _I, _F, _I, _I, _P],
+    "sprout_token_blend": [_P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P, _P],
+    "sprout_gated_group_norm": [_P, _P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _F, _I, _I, _P],
     "sprout_scaled_sum": [_P, _P, _F, _P, _F, _L, _P],
     "sprout_moe_route": [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _I, _I, _I, _I, _P],
     "sprout_exp_gates": [_P, _P, _I, _P, _P, _F, _I, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P],
     "sprout_exp_memory_out": [_P, _I, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P],
-    "sprout_unit_act": [_P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P],
+    "sprout_unit_act": [_P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P],
     "sprout_side_input_few": [_P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _F, _P, _P, _P],
     "sprout_side_gate": [_P, _I, _P, _I, _I, _P, _I, _P, _I, _I, _I, _P, _P],
     "sprout_rms_add": [_P, _P, _P, _I, _I, _F, _P],
@@ -349,7 +350,8 @@ def attention_simple(q, k_cache, v_cache, block_table, seq_of_token, positions, 
          k_cache.shape[0], _ptr(status, "status", torch.int32), _stream())
 
 
-def gemm_bf16(a, weight, out, status, bias=None, residual=None, orientation=0, split_k=1, swiglu=False, gate_activation="silu"):
+def gemm_bf16(a, weight, out, status, bias=None, residual=None, orientation=0, split_k=1, swiglu=False, gate_activation="silu",
+              groups=1, group_rows=0):
     """out = a @ weight.T (+ bias) (+ residual) on the tcgen05 tensor cores; a and weight bfloat16.
 
     ``residual`` must be ``out`` itself (float32): the product is added in place.  orientation 0
@@ -357,7 +359,9 @@ def gemm_bf16(a, weight, out, status, bias=None, residual=None, orientation=0, s
     tokens on M, 2 weights on M.  ``split_k`` > 1 divides K among CTAs (weights on M with a
     residual only; the partial sums are added with atomics).  ``swiglu``: weight rows interleave
     gate and up in blocks of 8 and ``out`` is bfloat16 [M, N/2] = act(gate) * up, act = ``gate_activation``: "silu" or
-    "gelu_tanh" (the tanh form of gelu)."""
+    "gelu_tanh" (the tanh form of gelu).  ``groups`` > 1: a is [M, groups * K], and output features [g * group_rows,
+    (g + 1) * group_rows) multiply its columns [g K, (g + 1) K) (the last group takes what is left): several matrices over
+    several inputs in one launch; ``group_rows`` is a multiple of 128."""
     if gate_activation not in ("silu", "gelu_tanh"):
         raise KernelError(f"gemm_bf16: the gated epilogue has silu and gelu_tanh, not {gate_activation!r}")
     _rows_contiguous(a, "a")
@@ -366,7 +370,8 @@ def gemm_bf16(a, weight, out, status, bias=None, residual=None, orientation=0, s
         raise KernelError("gemm_bf16: weight must be contiguous [N, K]")
     M, K = a.shape
     N = weight.shape[0]
-    if weight.shape[1] != K or tuple(out.shape) != (M, N // 2 if swiglu else N) or a.dtype != torch.bfloat16 \
+    K //= groups
+    if a.shape[1] != groups * K or weight.shape[1] != K or tuple(out.shape) != (M, N // 2 if swiglu else N) or a.dtype != torch.bfloat16 \
             or weight.dtype != torch.bfloat16:
         raise KernelError(f"gemm_bf16: shapes/dtypes do not fit: a {tuple(a.shape)} {a.dtype}, "
                           f"weight {tuple(weight.shape)} {weight.dtype}, out {tuple(out.shape)}")
@@ -376,7 +381,7 @@ def gemm_bf16(a, weight, out, status, bias=None, residual=None, orientation=0, s
         raise KernelError("gemm_bf16: the residual is added in place: pass out itself")
     _run("sprout_gemm_bf16", _ptr(a, "a"), _ptr(weight, "weight"), _ptr(bias, "bias", torch.float32, True),
          _ptr(out, "out"), _dtype_code(out.dtype), (3 if gate_activation == "gelu_tanh" else 2) if swiglu else (1 if residual is not None else 0), M, N, K, a.stride(0),
-         out.stride(0), orientation, split_k, _ptr(status, "status", torch.int32), _stream())
+         out.stride(0), orientation, split_k, int(groups), int(group_rows), _ptr(status, "status", torch.int32), _stream())
 
 
 def gemm_bf16_unscaled_supported(tokens: int, out_features: int, in_features: int, split_k: int) -> bool:
@@ -1023,11 +1028,12 @@ def headwise_gemm(a, weight, out, heads: int, a_head_stride: int, out_head_strid
          out_head_stride, _dtype_code(a.dtype), a.shape[0], heads, n, k, _stream())
 
 
-def latent_attention_simple(qlat, cache, block_table, seq_of_token, positions, sink, out, heads: int, rank: int, scale: float, status):
+def latent_attention_simple(qlat, cache, block_table, seq_of_token, positions, sink, out, heads: int, rank: int, scale: float, status,
+                            window: int = 0):
     """Causal attention of every (token, head) row of ``qlat`` [tokens, heads * width] over the rows of
     its request in ``cache`` [pages, 1, page_tokens, width]: score = scale * (row . key row), value = the
     key row's first ``rank`` elements; ``sink`` (float32 [heads] or None) adds exp(sink[h]) to the softmax
-    denominator.  out [tokens, heads * rank].  float32 arithmetic; the true 32-bit path."""
+    denominator; ``window`` > 0: a row sees its own position and the window - 1 before it.  out [tokens, heads * rank].  float32 arithmetic; the true 32-bit path."""
     T = qlat.shape[0]
     width = cache.shape[3]
     if cache.dim() != 4 or cache.shape[1] != 1 or not cache.is_contiguous() or cache.dtype != qlat.dtype or out.dtype != qlat.dtype \
@@ -1038,7 +1044,7 @@ def latent_attention_simple(qlat, cache, block_table, seq_of_token, positions, s
     _run("sprout_latent_attention_simple", _ptr(qlat, "qlat"), _ptr(cache, "cache"), _ptr(block_table, "block_table", torch.int32),
          block_table.stride(0), _ptr(seq_of_token, "seq_of_token", torch.int32), _ptr(positions, "positions", torch.int32),
          _ptr(sink, "sink", torch.float32, True), _ptr(out, "out"), _dtype_code(qlat.dtype), T, heads, width, rank,
-         cache.shape[2], cache.shape[0], float(scale), _ptr(status, "status", torch.int32), _stream())
+         cache.shape[2], cache.shape[0], float(scale), int(window), _ptr(status, "status", torch.int32), _stream())
 
 
 def latent_attention_mma_supported(width: int, rank: int) -> bool:
@@ -1066,7 +1072,7 @@ def latent_split_plan(requests: int, heads: int, rank: int, planned_keys: int, w
 
 
 def latent_attention_mma(qlat, cache, block_table, q_start, positions, context_lens, sink, out, heads: int, rank: int,
-                         scale: float, status, requests: int, splits: int = 0, split_keys: int = 0):
+                         scale: float, status, requests: int, splits: int = 0, split_keys: int = 0, window: int = 0):
     """The tensor-core form of ``latent_attention_simple`` (bfloat16).  ``splits`` 0: rows of any mix of
     portions and single tokens, 64 to a CTA.  ``splits`` >= 1: one token per request, its keys divided into
     ranges of ``split_keys`` that are merged through float32 scratch."""
@@ -1087,7 +1093,7 @@ def latent_attention_mma(qlat, cache, block_table, q_start, positions, context_l
          block_table.stride(0), _ptr(q_start, "q_start", torch.int32), _ptr(positions, "positions", torch.int32),
          _ptr(context_lens, "context_lens", torch.int32, True), _ptr(sink, "sink", torch.float32, True), _ptr(out, "out"),
          _ptr(scratch, "scratch", torch.float32, True), T, requests, heads, width, rank, cache.shape[2], cache.shape[0],
-         int(splits), int(split_keys), float(scale), _ptr(status, "status", torch.int32), _stream())
+         int(splits), int(split_keys), float(scale), int(window), _ptr(status, "status", torch.int32), _stream())
     if splits:
         global LAUNCHES
         LAUNCHES += 1                       # the merge kernel
@@ -1096,20 +1102,21 @@ def latent_attention_mma(qlat, cache, block_table, q_start, positions, context_l
 LATENT_ATTENTION = os.environ.get("SPROUT_LATENT_ATTENTION", "auto")      # "simple": the float32-arithmetic kernel for every step
 
 
-def latent_attention(qlat, cache, ctx, sink, out, heads: int, rank: int, scale: float, status):
+def latent_attention(qlat, cache, ctx, sink, out, heads: int, rank: int, scale: float, status, window: int = 0):
     """Latent attention of the step's rows over their requests' pages (``cache`` is a CacheView whose
     key buffer holds the rows).  float32 runs the plain kernel (the true 32-bit path), and so do sizes the
     tensor-core kernels do not take; bfloat16 runs the split-key kernel when every request brings one
-    token and the whole-rows kernel otherwise."""
+    token and the whole-rows kernel otherwise.  ``window`` > 0: a row sees its own position and the window - 1 before it."""
     width = cache.k.shape[3]
     if qlat.dtype != torch.bfloat16 or LATENT_ATTENTION == "simple" or not latent_attention_mma_supported(width, rank):
         return latent_attention_simple(qlat, cache.k, cache.block_table, ctx.seq_of_token, ctx.positions, sink, out, heads, rank,
-                                       scale, status)
+                                       scale, status, window=window)
     splits = split_keys = 0
     if ctx.max_q_len == 1:
-        splits, split_keys = latent_split_plan(ctx.num_seqs, heads, rank, ctx.planned_context or ctx.max_context, width)
+        planned = ctx.planned_context or ctx.max_context
+        splits, split_keys = latent_split_plan(ctx.num_seqs, heads, rank, min(planned, window) if window else planned, width)
     latent_attention_mma(qlat, cache.k, cache.block_table, ctx.q_start, ctx.positions, ctx.context_lens, sink, out, heads, rank,
-                         scale, status, ctx.num_seqs, splits, split_keys)
+                         scale, status, ctx.num_seqs, splits, split_keys, window=window)
 
 
 def depth_average(history, x, weights, n: int):
@@ -1122,11 +1129,11 @@ def depth_average(history, x, weights, n: int):
          _ptr(weights, "weights", torch.float32), int(n), x.numel(), _stream())
 
 
-def softcap(x, cap: float):
-    """x = cap * tanh(x / cap) in place (float32)."""
+def softcap(x, cap: float, factor: float = 1.0):
+    """x = cap * tanh(factor * x / cap) in place (float32); cap 0: x = factor * x."""
     if not x.is_contiguous():
         raise KernelError("softcap: x must be contiguous")
-    _run("sprout_softcap", _ptr(x, "x", torch.float32), float(cap), x.numel(), _stream())
+    _run("sprout_softcap", _ptr(x, "x", torch.float32), float(cap), float(factor), x.numel(), _stream())
 
 
 # ---------------------------------------------------------------------------------- layers wrapped in two norms, activations
@@ -1146,9 +1153,10 @@ def layernorm(x, gain, out, eps: float, rows=None, bias=None):
          _dtype_code(out.dtype), _ptr(rows, "rows", torch.int32, allow_none=True), R, H, float(eps), _stream())
 
 
-def norm_add(y, gain, x, eps: float, next_gain=None, h=None):
+def norm_add(y, gain, x, eps: float, next_gain=None, h=None, rms: bool = False, clear: bool = False):
     """x += layernorm(y) * gain (float32, in place); with ``next_gain`` and ``h`` also h = layernorm(x) * next_gain of
-    the new x, in h's dtype: the norm after a sublayer, the residual sum and the norm before the next sublayer."""
+    the new x, in h's dtype: the norm after a sublayer, the residual sum and the norm before the next sublayer.  ``rms``: RMS norms
+    instead of layer norms; ``clear``: y is left zeroed (the next sublayer adds into it)."""
     if y.dim() != 2 or not y.is_contiguous() or not x.is_contiguous() or x.shape != y.shape or gain.numel() != y.shape[1]:
         raise KernelError("norm_add: y and x must be contiguous [rows, width], gain [width]")
     if (next_gain is None) != (h is None) or (h is not None and (h.shape != x.shape or not h.is_contiguous()
@@ -1156,7 +1164,7 @@ def norm_add(y, gain, x, eps: float, next_gain=None, h=None):
         raise KernelError("norm_add: the next norm's gain and its output go together and have x's width")
     _run("sprout_norm_add", _ptr(y, "y", torch.float32), _ptr(gain, "gain", torch.float32), _ptr(x, "x", torch.float32),
          _ptr(next_gain, "next_gain", torch.float32, True), _ptr(h, "h", allow_none=True),
-         _dtype_code(h.dtype) if h is not None else F32, y.shape[0], y.shape[1], float(eps), _stream())
+         _dtype_code(h.dtype) if h is not None else F32, y.shape[0], y.shape[1], float(eps), 0 if rms else 1, 1 if clear else 0, _stream())
 
 
 def gated_rmsnorm(o, gain, gate, out, eps: float):
@@ -1192,7 +1200,7 @@ def glu_clamped(gate_up, out, limit: float, alpha: float):
 def rope_maps_append(rows, positions, seq_of_token, block_table, cos_table, sin_table, k_cache, v_cache, q_vectors: int,
                      kv_heads: int, maps: int, dim: int, vdim: int, page_tokens: int, write: bool, status,
                      unit_eps: float = 0.0, value_from_key: bool = False, q_weight=None, k_weight=None, weight_eps: float = 0.0,
-                     interleaved: bool = False, value_turn=None):
+                     interleaved: bool = False, value_turn=None, growth=None):
     """Rotate the first ``2 * cos_table.shape[1]`` elements of every query vector (in place) and key vector by the token's
     position, in half-split pairs or, with ``interleaved``, in pairs (2i, 2i + 1); append keys ([pages, kv_heads, page_tokens, maps * dim]) and values
     ([pages, kv_heads, page_tokens, vdim]) when ``write``.  A row holds q_vectors * dim query elements, then (when
@@ -1203,7 +1211,9 @@ def rope_maps_append(rows, positions, seq_of_token, block_table, cos_table, sin_
     ``dim`` (``weight_eps`` inside the root) and multiplied by the weight; weights as wide as all query vectors and all key
     vectors together ([q_vectors * dim] and [kv_heads * maps * dim]): the norm is over the token's whole projection instead.
     ``value_turn`` = (cos, sin), tables [max_positions, vdim / 2]: value rows are turned by the token's position over all of
-    their elements before they are cached, in pairs like the keys'."""
+    their elements before they are cached, in pairs like the keys'.  ``growth`` = (coef, every): query vectors at position p are
+    multiplied by 1 + coef * ln(floor((p + 1) / every) + 1), after norm and rotation."""
+    growth_coef, growth_every = (0.0, 0) if growth is None else (float(growth[0]), int(growth[1]))
     _rows_contiguous(rows, "rows")
     weights = [(w, width) for w, width in ((q_weight, q_vectors * dim), (k_weight, kv_heads * maps * dim)) if w is not None]
     whole = all(w.numel() == width for w, width in weights) and any(w.numel() != dim for w, _ in weights)
@@ -1230,7 +1240,7 @@ def rope_maps_append(rows, positions, seq_of_token, block_table, cos_table, sin_
          kv_heads, maps, dim, rot, vdim, page_tokens, k_cache.shape[0] if write else 1, 1 if write else 0,
          float(unit_eps), 1 if value_from_key else 0, _ptr(q_weight, "q_weight", torch.float32, True),
          _ptr(k_weight, "k_weight", torch.float32, True), float(weight_eps), 1 if whole else 0, 1 if interleaved else 0, v_cos, v_sin,
-         _ptr(status, "status", torch.int32), _stream())
+         growth_coef, growth_every, _ptr(status, "status", torch.int32), _stream())
 
 
 MASK_KINDS = {"causal": 0, "window": 1, "chunk": 2}
@@ -1550,7 +1560,7 @@ def _scan_view(t, name: str, width: int, dtype):
 
 def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: int, vdim: int, status, per_head: bool = False,
                tau: float = 1.0, q_scale: float = 1.0, a_log=None, skip=None, given=None, ones_col: bool = False, floor=None,
-               q_silu: bool = False):
+               q_silu: bool = False, bonus=None):
     """Per request and head, token by token: S = diag(a) S + (c k) v^T, o = S^T (q_scale q) + skip_h v, the state float32
     [slots, heads, dim, vdim] read and written at the requests' slots (``state``: a ``StateView``-like with ``buffer`` and
     ``slots``).  q, k [tokens, groups * dim] (heads of a group share them), v [tokens, heads * vdim], views with unit inner
@@ -1558,6 +1568,8 @@ def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: 
     ``per_head``: z [tokens, heads], dt = softplus(z + bias), a = exp(-exp(a_log) dt) for all of the head's channels, c = dt.
     ``floor`` (float32 [heads * dim]): z [tokens, heads * dim], a = floor + (1 - floor) sigmoid(z + bias) and 1 - a takes the place
     of c k (``k`` is None); with ``q_silu`` q passes silu first (in this form only).
+    ``bonus`` (float32 [heads * dim]): z [tokens, heads * dim], a = exp(-exp(z + bias)), c = 1, and the output reads the state before the
+    token plus the token's own write weighed by the bonus: o = (S_before + diag(bonus) k v^T)^T (q_scale q).
     ``given`` = (a, c), float32 [tokens, heads] each: the decay and the factor on k per head, ready-made (z and bias are None).
     ``ones_col``: the value rows are narrower than the state, v [tokens, heads * v_cols] with v_cols < vdim, and the state's
     column v_cols is fed the constant 1 as a value (the columns after it 0): that column of the state is then the sum of the
@@ -1573,6 +1585,9 @@ def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: 
     if (k is None) != (floor is not None) or (floor is not None and (floor.dtype != torch.float32 or floor.numel() != heads * dim
                                                                      or groups != heads or per_head or given is not None)):
         raise KernelError("gated_scan: a forget gate with a floor has no keys, float32 floors [heads * dim] and query vectors per head")
+    if bonus is not None and (bonus.dtype != torch.float32 or bonus.numel() != heads * dim or groups != heads or per_head or given is not None
+                              or floor is not None):
+        raise KernelError("gated_scan: a bonus is float32 [heads * dim], with vectors and decays per head and channel")
     k_ptr, k_stride = (None, 0) if k is None else _scan_view(k, "k", groups * dim, dtype)
     v_ptr, v_stride = _scan_view(v, "v", heads * v_cols, dtype)
     if given is not None:
@@ -1608,7 +1623,7 @@ def gated_scan(q, k, v, z, bias, ctx, state, out, heads: int, groups: int, dim: 
         da, dc = given
     _run("sprout_gated_scan", q_ptr, q_stride, k_ptr, k_stride, v_ptr, v_stride, z_ptr, z_stride, 1 if z_f32 else 0,
          _dtype_code(dtype), _ptr(bias, "bias", torch.float32, True), _ptr(a_log if floor is None else floor, "a_log", torch.float32, True), _ptr(skip, "skip", torch.float32, True),
-         1.0 / float(tau), float(q_scale), 2 if given is not None else 3 if floor is not None else 1 if per_head else 0, state.slots.numel(), heads, groups, dim, vdim,
+         _ptr(bonus, "bonus", torch.float32, True), 1.0 / float(tau), float(q_scale), 2 if given is not None else 3 if floor is not None else 4 if bonus is not None else 1 if per_head else 0, state.slots.numel(), heads, groups, dim, vdim,
          _ptr(ctx.q_start, "q_start", torch.int32), _ptr(state.slots, "state_slots", torch.int32),
          _ptr(buffer, "state", torch.float32), buffer.shape[0], _ptr(out, "out", torch.float32),
          _ptr(status, "status", torch.int32), tokens, SCAN_CHUNK, max_chunks, _ptr(da, "decays", torch.float32, True),
@@ -1675,20 +1690,38 @@ def causal_conv(rows, weight, bias, out, ctx, state, status, silu: bool = True):
          1 if silu else 0, _ptr(status, "status", torch.int32), _stream())
 
 
+def token_blend(h, mu, out, ctx, state, status):
+    """out[t, s] = h[t] + (h[t - 1] - h[t]) * mu[s]: ``mu`` float32 [parts, width] blends of every row with the row before it,
+    out [tokens, parts * width] of h's dtype.  The row before a request's first token of the step is its row of ``state``
+    (float32 [slots, width]; zeros for a new sequence), which is replaced by the request's last row."""
+    tokens, width = h.shape
+    parts = mu.shape[0]
+    buffer = state.buffer
+    if not h.is_contiguous() or not out.is_contiguous() or out.dtype != h.dtype or tuple(out.shape) != (tokens, parts * width) \
+            or tuple(mu.shape) != (parts, width) or not mu.is_contiguous():
+        raise KernelError("token_blend: h must be contiguous [tokens, width], mu [parts, width], out [tokens, parts * width]")
+    if buffer.dtype != torch.float32 or not buffer.is_contiguous() or tuple(buffer.shape[1:]) != (width,):
+        raise KernelError("token_blend: state must be contiguous float32 [slots, width]")
+    _run("sprout_token_blend", _ptr(h, "h"), _ptr(mu, "mu", torch.float32), _ptr(out, "out"), _dtype_code(h.dtype),
+         _ptr(ctx.q_start, "q_start", torch.int32), _ptr(ctx.seq_of_token, "seq_of_token", torch.int32),
+         _ptr(state.slots, "state_slots", torch.int32), _ptr(buffer, "state", torch.float32), buffer.shape[0], tokens, width, parts,
+         _ptr(status, "status", torch.int32), _stream())
+
+
 def gated_group_norm(o, gate, weight, out, eps: float, groups: int = 1, gate_first: bool = False, silu: bool = True):
     """Rows of ``o`` (float32 [rows, width]) in ``groups`` equal parts, each divided by its root mean square (eps inside
     the root), times ``weight`` (float32; it repeats every weight.numel() elements: a weight per head, or one for the whole
     row), times act(gate), act = silu or sigmoid; with ``gate_first`` the gate is applied before the norm.  ``gate`` is a
-    [rows, width] view with unit inner stride of out's dtype, or None (no gate)."""
+    [rows, width] view with unit inner stride of out's dtype or float32, or None (no gate)."""
     if gate is not None:
         _rows_contiguous(gate, "gate")
     rows, width = o.shape
     if not o.is_contiguous() or o.dtype != torch.float32 or not out.is_contiguous() or out.shape != o.shape \
-            or (gate is not None and (gate.shape != o.shape or gate.dtype != out.dtype)) or (gate is None and gate_first) \
+            or (gate is not None and (gate.shape != o.shape or gate.dtype not in (out.dtype, torch.float32))) or (gate is None and gate_first) \
             or width % weight.numel() or width % groups:
         raise KernelError("gated_group_norm: shapes or dtypes do not fit")
     _run("sprout_gated_group_norm", _ptr(o, "o", torch.float32), _ptr(gate, "gate", allow_none=True), 0 if gate is None else gate.stride(0),
-         _ptr(weight, "weight", torch.float32), weight.numel(), _ptr(out, "out"), _dtype_code(out.dtype), rows, width,
+         _dtype_code(out.dtype if gate is None else gate.dtype), _ptr(weight, "weight", torch.float32), weight.numel(), _ptr(out, "out"), _dtype_code(out.dtype), rows, width,
          int(groups), float(eps), 1 if gate_first else 0, 1 if silu else 0, _stream())
 
 
@@ -1742,22 +1775,22 @@ def exp_memory_out(o, m, gate, weight, out, heads: int, vdim: int, eps: float, o
 
 # ---------------------------------------------------------------------------------- rows of feed-forwards and of inputs to the stream
 
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu_erf": 2}
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu_erf": 2, "tanh": 3}
 
 
 def unit_act(rows, out, activation: str, gated: bool, row_logits=None):
     """out = act(gate) * up for rows [gate: ff | up: ff] (``gated``), or act(rows) for rows of ff elements; ``rows`` and
-    ``out`` are views with unit inner stride of one dtype.  ``row_logits`` (a float32 view with one number per row): row r is
+    ``out`` are views with unit inner stride of one dtype, or float32 ``rows`` beside a bfloat16 ``out``.  ``row_logits`` (a float32 view with one number per row): row r is
     also multiplied by sigmoid(row_logits[r])."""
     _rows_contiguous(rows, "rows")
     _rows_contiguous(out, "out")
     ff = out.shape[1]
-    if activation not in ACTIVATIONS or rows.dtype != out.dtype or rows.shape[0] != out.shape[0] or rows.shape[1] < (2 if gated else 1) * ff:
+    if activation not in ACTIVATIONS or rows.dtype not in (out.dtype, torch.float32) or rows.shape[0] != out.shape[0] or rows.shape[1] < (2 if gated else 1) * ff:
         raise KernelError("unit_act: shapes, dtypes or the activation's name do not fit")
     if row_logits is not None and (row_logits.dtype != torch.float32 or row_logits.shape[0] != out.shape[0]):
         raise KernelError("unit_act: one float32 logit per row")
-    _run("sprout_unit_act", rows.data_ptr(), rows.stride(0), out.data_ptr(), out.stride(0), _dtype_code(out.dtype), out.shape[0], ff,
-         ACTIVATIONS[activation], 1 if gated else 0, None if row_logits is None else row_logits.data_ptr(),
+    _run("sprout_unit_act", rows.data_ptr(), rows.stride(0), _dtype_code(rows.dtype), out.data_ptr(), out.stride(0), _dtype_code(out.dtype),
+         out.shape[0], ff, ACTIVATIONS[activation], 1 if gated else 0, None if row_logits is None else row_logits.data_ptr(),
          0 if row_logits is None else row_logits.stride(0), _stream())
 
 

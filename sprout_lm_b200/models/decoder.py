@@ -138,6 +138,11 @@ class DecoderModel:
                 block.forward(x, ctx, cache, state, primed=primed, finish=finish)
                 primed = ahead
                 continue
+            if self.stream is None and getattr(block, "chains", False):
+                # a block whose last step is a norm may make the next block's input in the same launch
+                following = self.blocks[self.spec.order[n + 1].layer] if n + 1 < len(self.spec.order) else None
+                primed = block.forward(x, ctx, cache, state, primed=primed, following=following)
+                continue
             block.forward(x, ctx, cache, state)
             primed = None
             if self.stream:

@@ -125,9 +125,13 @@ class PostNormBlock(Part):
 @register_part("block", "sandwich_norm")
 class SandwichNormBlock(Part):
     """A norm before and after each sublayer: x += norm_1(mixer(norm_0(x))), then x += norm_3(ffn(norm_2(x))).
+    The norms are layer norms or RMS norms, all of a block alike.
     The stream and the sums are float32.  A layer without a feed-forward (``feed_forward.kind == "none"``) has the
     first two norms only.  A sublayer adds its output into a zeroed float32 buffer; one kernel then norms that
-    buffer, adds it to the stream and, after the mixer, also makes what the feed-forward reads."""
+    buffer, adds it to the stream, clears the buffer for the next sublayer and makes what that one reads.  That goes on
+    from block to block: ``forward`` takes ``primed`` = (h, y), what the block before left (the first sublayer's input and
+    the zeroed buffer), and returns the same for ``following``, the next block, or None."""
+    chains = True
 
     def __init__(self, prefix: str, layer: LayerSpec):
         self.has_ffn = layer.feed_forward.kind != "none"
@@ -135,8 +139,9 @@ class SandwichNormBlock(Part):
             raise ValueError("a sandwich_norm block has two norms per sublayer")
         self.norms = [build_part("norm", spec, prefix) for spec in layer.norms]
         for norm in self.norms:
-            if getattr(norm, "fused_kind", None) != "layernorm":
-                raise ValueError("a sandwich_norm block takes layer norms")
+            if getattr(norm, "fused_kind", None) not in ("layernorm", "rmsnorm") or norm.fused_kind != self.norms[0].fused_kind:
+                raise ValueError("a sandwich_norm block takes layer norms or RMS norms, all alike")
+        self.rms = self.norms[0].fused_kind == "rmsnorm"
         self.mixer = build_part("mixer", layer.mixer, prefix)
         self.feed_forward = build_part("feed_forward", layer.feed_forward, prefix) if self.has_ffn else None
 
@@ -151,24 +156,29 @@ class SandwichNormBlock(Part):
             part.load(source)
         self.dtype = source.runtime.dtype
 
-    def forward(self, x, ctx, cache, state):
+    def _close(self, y, x, after, following):
+        """x += after(y); with a norm ``following`` y is cleared and that norm's output of the new x returned."""
         import torch
         from .. import kernels
-        before, after = self.norms[0], self.norms[1]
-        y = torch.zeros_like(x)
-        self.mixer.forward(before.forward(x), y, ctx, cache, state)
-        if not self.has_ffn:
-            kernels.norm_add(y, after.gain, x, after.eps)
-            return
-        if self.norms[2].eps == after.eps:
-            h = torch.empty(x.shape, dtype=self.dtype, device=x.device)
-            kernels.norm_add(y, after.gain, x, after.eps, next_gain=self.norms[2].gain, h=h)
-        else:
-            kernels.norm_add(y, after.gain, x, after.eps)
-            h = self.norms[2].forward(x)
-        y.zero_()
-        self.feed_forward.forward(h, y, ctx)
-        kernels.norm_add(y, self.norms[3].gain, x, self.norms[3].eps)
+        if following is None:
+            kernels.norm_add(y, after.gain, x, after.eps, rms=self.rms)
+            return None
+        if following.eps != after.eps or getattr(following, "bias", None) is not None:
+            kernels.norm_add(y, after.gain, x, after.eps, rms=self.rms, clear=True)
+            return following.forward(x)
+        h = torch.empty(x.shape, dtype=self.dtype, device=x.device)
+        kernels.norm_add(y, after.gain, x, after.eps, next_gain=following.gain, h=h, rms=self.rms, clear=True)
+        return h
+
+    def forward(self, x, ctx, cache, state, primed=None, following=None):
+        import torch
+        h, y = primed if primed is not None else (self.norms[0].forward(x), torch.zeros_like(x))
+        last = following.norms[0] if isinstance(following, SandwichNormBlock) and following.rms == self.rms else None
+        self.mixer.forward(h, y, ctx, cache, state)
+        if self.has_ffn:
+            self.feed_forward.forward(self._close(y, x, self.norms[1], self.norms[2]), y, ctx)
+        h = self._close(y, x, self.norms[-1], last)
+        return None if h is None else (h, y)
 
 
 @register_part("block", "parallel_residual")

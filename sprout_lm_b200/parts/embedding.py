@@ -1,6 +1,6 @@
 """Token embedding (a row copy, src/qwen.ts:162-163; ``scale`` multiplies the rows when a model asks for it) and the output head
 (logits = W h, no bias; W is the embedding matrix itself when tied: src/qwen.ts:152,203).
-With ``softcap`` the head's logits become softcap * tanh(logits / softcap)."""
+With ``scale`` the head's logits are multiplied by it, with ``softcap`` they then become softcap * tanh(logits / softcap)."""
 from __future__ import annotations
 
 import torch
@@ -72,12 +72,12 @@ class TokenPairEmbedding(TokenEmbedding):
 class LMHead(Part):
     def __init__(self, prefix: str, vocab_size: int, hidden_size: int, tied_to: str | None = None,
                  name: str = "lm_head", suffix: str = ".weight", softcap: float | None = None,
-                 any_inner_size: bool = False):
+                 any_inner_size: bool = False, scale: float = 1.0):
         if softcap is not None and not softcap > 0:
             raise ValueError("lm_head: softcap must be positive")
         self.vocab_size, self.hidden_size = vocab_size, hidden_size
         self.softcap = None if softcap is None else float(softcap)
-        self.any_inner_size = any_inner_size
+        self.any_inner_size, self.scale = any_inner_size, float(scale)
         self.tensor_name = f"{prefix}{tied_to or name}{suffix}"
         self.tied = tied_to is not None
         self.linear = None
@@ -90,6 +90,6 @@ class LMHead(Part):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         logits = self.linear.forward(h, out_dtype=torch.float32)
-        if self.softcap is not None:
-            kernels.softcap(logits, self.softcap)
+        if self.softcap is not None or self.scale != 1.0:
+            kernels.softcap(logits, self.softcap or 0.0, factor=self.scale)
         return logits

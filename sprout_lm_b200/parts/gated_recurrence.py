@@ -22,6 +22,15 @@ f = lower + (1 - lower) sigmoid(W_f h + b_f) (heads x dim); a = f, and c k = 1 -
 key.  Each head's o is divided by its root mean square over value_dim and multiplied by a weight [value_dim] that the heads
 share; the heads side by side are projected by W_o.
 
+``rwkv_time_mixing`` (the RWKV recurrence with a decay made from the input): with h' the row before (zeros ahead of the first), each of
+five inputs is a blend of its own, h + (h' - h) * mu_s; r, k, v = W_s of their blends (heads x dim each), gate = silu(W_g of its
+blend), and a decay per head and channel, a = exp(-exp(W_w2 tanh(W_w1 of its blend) + w0)).  o_t reads the state before the token
+and the token's own write weighed by a learned bonus u per head and channel: o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, then
+S_t = diag(a_t) S_(t-1) + k_t v_t^T.  Each head's o is divided by its root mean square over dim; the heads side by side are
+multiplied by a weight [heads * dim] and by the gate and projected by W_o.  The request's last row is a second state tensor.
+The projections leave their products in float32, so nothing that enters the recurrence is rounded to 16 bits but its
+matrix products' inputs.
+
 ``out_scale`` multiplies the mixer's output (it is folded into the norm's weight), so that a block that runs several
 mixers side by side can weigh them without a kernel of its own.
 """
@@ -31,7 +40,7 @@ import torch
 
 from .. import kernels
 from .base import Part, StateSpec, StateView, TensorDecl, WeightSource, register_part
-from .linear import Linear
+from .linear import GroupedLinear, Linear
 
 
 @register_part("mixer", "gated_linear_attention")
@@ -208,3 +217,68 @@ class ForgetWriteAttention(Part):
         normed = torch.empty((rows.shape[0], vw), dtype=rows.dtype, device=rows.device)
         kernels.gated_group_norm(o, None, self.gain, normed, self.eps, groups=self.heads)
         self.out.forward(normed, residual=x)
+
+
+@register_part("mixer", "rwkv_time_mixing")
+class RWKVTimeMixing(Part):
+    BLENDS = ("r", "k", "v", "g", "w")
+    DEFAULT_NAMES = {"r": "r", "k": "k", "v": "v", "g": "g", "w1": "w1", "w2": "w2", "w0": "w0", "u": "u", "norm": "norm", "o": "o",
+                     **{"mu_" + key: "mu." + key for key in BLENDS}}
+
+    def __init__(self, prefix: str, hidden_size: int, heads: int, dim: int, eps: float, decay_rank: int | None = None,
+                 out_scale: float = 1.0, stem: str = "", names: dict | None = None):
+        """``stem`` stands between the prefix and every tensor's name; ``decay_rank`` None: the decay's inner size is whatever the
+        checkpoint's tensors have."""
+        if hidden_size <= 0 or heads <= 0 or dim <= 0 or eps <= 0:
+            raise ValueError("rwkv_time_mixing: sizes and eps must be positive")
+        if decay_rank is not None and decay_rank <= 0:
+            raise ValueError("rwkv_time_mixing: the decay's inner size must be positive")
+        self.hidden_size, self.heads, self.dim, self.eps, self.out_scale = hidden_size, heads, dim, float(eps), float(out_scale)
+        self.decay_rank = decay_rank
+        self.names = {key: prefix + stem + value for key, value in {**self.DEFAULT_NAMES, **(names or {})}.items()}
+        self.runtime = None
+
+    def cache_spec(self):
+        return None
+
+    def state_spec(self):
+        return (StateSpec(shape=(self.hidden_size,), dtype=torch.float32),
+                StateSpec(shape=(self.heads, self.dim, self.dim), dtype=torch.float32))
+
+    def tensor_decls(self):
+        n, width, rank = self.names, self.heads * self.dim, self.decay_rank
+        return [*(TensorDecl(n["mu_" + key], (self.hidden_size,), "share") for key in self.BLENDS),
+                *(TensorDecl(n[key], (width, self.hidden_size)) for key in ("r", "k", "v", "g")),
+                TensorDecl(n["w1"], (rank, self.hidden_size)), TensorDecl(n["w2"], (width, rank)), TensorDecl(n["w0"], (width,), "bias"),
+                TensorDecl(n["u"], (self.heads, self.dim), "wide"), TensorDecl(n["norm"], (width,), "gain"),
+                TensorDecl(n["o"], (self.hidden_size, width))]
+
+    def load(self, source: WeightSource):
+        n, status = self.names, source.runtime.status
+        self.runtime = source.runtime
+        if source.raw(n["w1"]).shape[0] != source.raw(n["w2"]).shape[1]:
+            raise ValueError("rwkv_time_mixing: the decay's two matrices do not fit each other")
+        self.blend = torch.stack([source.vector(n["mu_" + key]) for key in self.BLENDS]).contiguous()
+        self.proj = GroupedLinear([source.to_device_matrix(source.raw(n[key])) for key in ("r", "k", "v", "g", "w1")], status)
+        self.decay_out = Linear(source.matrix(n["w2"]), None, status, any_inner_size=True)
+        self.decay_bias, self.bonus = source.vector(n["w0"]), source.vector(n["u"]).reshape(-1).contiguous()
+        self.gain = (source.vector(n["norm"]) * self.out_scale).contiguous()
+        self.out = Linear(source.matrix(n["o"]), None, status, any_inner_size=True)
+
+    def forward(self, h, x, ctx, cache, state: StateView):
+        """x (float32) += out_scale * W_o (per-head o / rms(o) * w * gate); the requests' states advance."""
+        if state is None:
+            raise RuntimeError("rwkv_time_mixing: the layer needs a state slot per request")
+        status, tokens, width = self.runtime.status, h.shape[0], self.heads * self.dim
+        blended = torch.empty((tokens, len(self.BLENDS) * self.hidden_size), dtype=h.dtype, device=h.device)
+        kernels.token_blend(h, self.blend, blended, ctx, state.part(0), status)
+        r, k, v, gate, inner = self.proj.forward_float32(blended)
+        low = torch.empty(inner.shape, dtype=h.dtype, device=h.device)
+        kernels.unit_act(inner, low, "tanh", gated=False)
+        z = self.decay_out.forward_float32(low)
+        o = torch.empty((tokens, width), dtype=torch.float32, device=h.device)
+        kernels.gated_scan(r, k, v, z, self.decay_bias, ctx, state.part(1), o, self.heads, self.heads, self.dim, self.dim, status,
+                           bonus=self.bonus)
+        gated = torch.empty((tokens, width), dtype=h.dtype, device=h.device)
+        kernels.gated_group_norm(o, gate, self.gain, gated, self.eps, groups=self.heads, silu=True)
+        self.out.forward(gated, residual=x)

@@ -2,7 +2,9 @@
 all heads, c = RMSNorm(W_dkv h)[:rank] * w and k_rot = the last ``rot_dim`` outputs of W_dkv h rotated by
 the token's position.  Head n's key is [W_uk,n c | k_rot], its value W_uv,n c, its query
 [q_n (dim, unrotated) | q_rot,n (rot_dim, rotated)]; the score is scale * (q_n . W_uk,n c + q_rot,n . k_rot),
-the mask causal, and the softmax's denominator may hold one more term exp(sink_n) per head.
+the mask causal or (``window``) a sliding window of that many positions, a query's own included, and the softmax's denominator
+may hold one more term exp(sink_n) per head.  With a window the cache slot is of kind ``window``: pages that no later query
+can see are given back.
 
 The up-projections are folded to the query's side, so that nothing per head is ever made of the cache:
 q_lat,n = W_uk,n^T q_n (rank wide), score = scale * ([q_lat,n | q_rot,n] . [c | k_rot]), the weighted sum of
@@ -30,12 +32,17 @@ DEFAULT_NAMES = {"q": "q", "dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": 
 class LatentAttention(Part):
     def __init__(self, prefix: str, hidden_size: int, heads: int, dim: int, rot_dim: int, value_dim: int, kv_rank: int,
                  scale: float, eps: float, position: PartSpec, q_rank: int | None = None, own_kv: bool = True,
-                 sink: bool = True, names: dict | None = None):
+                 sink: bool = True, names: dict | None = None, window: int | None = None):
         for label, value in (("hidden_size", hidden_size), ("heads", heads), ("value_dim", value_dim), ("kv_rank", kv_rank)):
             if value <= 0:
                 raise ValueError(f"latent_attention: {label} must be positive (got {value})")
         if dim < 0 or rot_dim < 0 or dim + rot_dim == 0:
             raise ValueError("latent_attention: a head needs unrotated or rotated query/key dimensions")
+        if window is not None and window <= 0:
+            raise ValueError("latent_attention: a window has at least one position")
+        if scale <= 0:
+            raise ValueError("latent_attention: scale must be positive")
+        self.window = window
         if q_rank is not None and q_rank <= 0:
             raise ValueError("latent_attention: q_rank must be positive when given")
         self.hidden_size, self.heads, self.dim, self.rot_dim = hidden_size, heads, dim, rot_dim
@@ -48,14 +55,16 @@ class LatentAttention(Part):
 
     # ---- what it keeps: one row per token, no values of their own
     def cache_spec(self):
-        return CacheSpec(kv_heads=1, head_dim=self.width, kind="full", value_dim=0)
+        return CacheSpec(kv_heads=1, head_dim=self.width, kind="full" if self.window is None else "window", window=self.window,
+                         value_dim=0)
 
     def state_spec(self):
         return None
 
     def decode_plan(self, requests: int, max_keys: int, planned_context: int, page_tokens: int):
         """How a step of one token per request divides its keys among CTAs: it follows the contexts' length."""
-        return kernels.latent_split_plan(requests, self.heads, self.kv_rank, planned_context, self.width)
+        keys = planned_context if self.window is None else min(planned_context, self.window)
+        return kernels.latent_split_plan(requests, self.heads, self.kv_rank, keys, self.width)
 
     # ---- weights
     def tensor_decls(self):
@@ -124,7 +133,8 @@ class LatentAttention(Part):
         kernels.latent_query_tail(q, q_lat, ctx.positions, cos, sin, self.interleaved, self.heads, self.dim, self.rot_dim,
                                   self.kv_rank, status)
         mixed = torch.empty((tokens, self.heads * self.kv_rank), dtype=h.dtype, device=h.device)
-        kernels.latent_attention(q_lat, cache, ctx, self.sink, mixed, self.heads, self.kv_rank, self.scale, status)
+        kernels.latent_attention(q_lat, cache, ctx, self.sink, mixed, self.heads, self.kv_rank, self.scale, status,
+                                 window=self.window or 0)
         attended = torch.empty((tokens, self.heads * self.value_dim), dtype=h.dtype, device=h.device)
         kernels.headwise_gemm(mixed, self.uv, attended, self.heads, self.kv_rank, self.value_dim)
         self.out.forward(attended, residual=x)

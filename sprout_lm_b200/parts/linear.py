@@ -32,6 +32,43 @@ def small_batch_split_k(out_features: int, in_features: int, tokens: int, residu
     return max(1, min(k_blocks, sms // tiles))
 
 
+class GroupedLinear:
+    """Several matrices over inputs of their own, y_g = W_g a_g: the inputs stand side by side in ``a``'s rows
+    [tokens, groups * K], the weights are [rows_g, K].  On the tensor cores, where all matrices but the last have one
+    number of rows that fills whole tiles, they are one product in one launch; otherwise a product each."""
+    TILE = 128
+
+    def __init__(self, weights, status: torch.Tensor):
+        weights = list(weights)
+        self.rows = [w.shape[0] for w in weights]
+        self.inner, self.status = weights[0].shape[1], status
+        first = self.rows[0]
+        self.fused = None
+        if weights[0].dtype == torch.bfloat16 and weights[0].is_cuda and self.inner % 8 == 0 and len(weights) > 1 and first % self.TILE == 0 \
+                and all(r == first for r in self.rows[:-1]):
+            whole = torch.cat(weights, dim=0)
+            pad = -whole.shape[0] % (256 if first % 256 == 0 else 8)      # CTA pairs take 256 features each
+            self.fused = torch.nn.functional.pad(whole, (0, 0, 0, pad)).contiguous()
+            self.sms = kernels.sm_count(whole.device)
+            return
+        self.parts = [Linear(w.contiguous(), None, status, any_inner_size=True) for w in weights]
+
+    def forward_float32(self, a: torch.Tensor) -> list:
+        """[W_0 a_0, W_1 a_1, ...] as float32 views [tokens, rows_g]."""
+        if self.fused is None:
+            return [part.forward_float32(a[:, g * self.inner:(g + 1) * self.inner]) for g, part in enumerate(self.parts)]
+        tokens, features = a.shape[0], self.fused.shape[0]
+        few = tokens <= 256                # K split among CTAs that add into a zeroed buffer, so that every SM streams a share
+        out = (torch.zeros if few else torch.empty)((tokens, features), dtype=torch.float32, device=a.device)
+        kernels.gemm_bf16(a, self.fused, out, self.status, residual=out if few else None, groups=len(self.rows), group_rows=self.rows[0],
+                          split_k=small_batch_split_k(features, self.inner, tokens, True, self.sms) if few else 1)
+        at, views = 0, []
+        for rows in self.rows:
+            views.append(out[:, at:at + rows])
+            at += rows
+        return views
+
+
 class Linear:
     def __init__(self, weight: torch.Tensor, bias: torch.Tensor | None, status: torch.Tensor, any_inner_size: bool = False):
         self.weight = weight

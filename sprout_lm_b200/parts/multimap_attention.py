@@ -25,7 +25,8 @@ denominator (a sink whose score is 0, without a tensor); ``conv``: the projectio
 that many taps (no bias, zeros before the start; the matrix's name + ".conv", [channels, taps]) before norm and rotation, and
 its last taps - 1 inputs are a per-request state; ``value_position`` (a ``position`` PartSpec over ``value_dim``, pairs laid
 out like the keys'): value rows are cached turned by their position, and every head's output is turned back by the query's
-position before the gate; ``out_scale`` multiplies the heads' output; ``value_from_key``: there is no value projection, the value row
+position before the gate; ``query_growth`` = (coef, every): after norm and rotation a query at position p is multiplied by
+1 + coef ln(floor((p + 1) / every) + 1); ``out_scale`` multiplies the heads' output; ``value_from_key``: there is no value projection, the value row
 is the key row as projected, before rotation and norm (``value_dim`` = ``maps * dim``).
 
 A layer may read the keys and values another layer cached (its run-order entry has ``writes_cache=False``): it then
@@ -55,7 +56,7 @@ class MultiMapAttention(Part):
                  own_kv: bool = True, names: dict | None = None, mask=None, sink: bool = False, gate=False,
                  unit_norm_eps: float = 0.0, value_from_key: bool = False, softcap: float = 0.0, bias: bool = False,
                  qk_norm_eps: float = 0.0, qk_norm_span: str = "vector", unit_sink: bool = False, conv: int | None = None,
-                 value_position: PartSpec | None = None):
+                 value_position: PartSpec | None = None, query_growth=None):
         if heads <= 0 or kv_heads <= 0 or heads % kv_heads:
             raise ValueError(f"multimap_attention: heads ({heads}) must be a positive multiple of kv_heads ({kv_heads})")
         if maps not in (1, 2):
@@ -86,6 +87,9 @@ class MultiMapAttention(Part):
             raise ValueError("multimap_attention: convolutions, turned values and element gates are for one map per head with values of its own")
         if conv is not None and (conv < 1 or bias):
             raise ValueError("multimap_attention: a convolution has at least one tap and stands on projections without biases")
+        if query_growth is not None and (int(query_growth[1]) != query_growth[1] or query_growth[1] <= 0):
+            raise ValueError("multimap_attention: the queries' growth counts positions in whole, positive steps")
+        self.query_growth = None if query_growth is None else (float(query_growth[0]), int(query_growth[1]))
         self.mask, self.has_sink, self.has_gate = mask, bool(sink), bool(gate)
         self.gate_width = heads * value_dim if gate == "element" else heads
         self.norm_whole, self.unit_sink, self.conv = qk_norm_span == "projection", bool(unit_sink), conv
@@ -212,7 +216,7 @@ class MultiMapAttention(Part):
                                  self.heads * self.maps, self.kv_heads, self.maps, self.dim, self.value_dim, cache.page_tokens,
                                  cache.write, status, unit_eps=self.unit_norm_eps, value_from_key=self.value_from_key,
                                  q_weight=self.q_norm, k_weight=self.k_norm, weight_eps=self.qk_norm_eps,
-                                 interleaved=self.interleaved, value_turn=self.turn)
+                                 interleaved=self.interleaved, value_turn=self.turn, growth=self.query_growth)
         attended = torch.empty((rows.shape[0], self.heads * self.value_dim), dtype=rows.dtype, device=rows.device)
         kernels.multimap_attention(rows[:, :self.q_width], cache, ctx, attended, self.heads, self.kv_heads, self.maps, self.dim,
                                    self.value_dim, self.scale, self.lam, self.norm_eps, self.out_scale, status, mask=self.mask,
