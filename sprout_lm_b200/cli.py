@@ -106,6 +106,21 @@ TINY_CONFIGS["Z"] = {
                                  "right": {"heads": 2, "kv_heads": 2, "dim": 16, "vdim": 64, "conv": 2}, "right_scale": 1.0}))]}
 
 
+# --tiny W: a tiny random Buzinex model (latent attention over two windows, attention with queries that grow and capped scores,
+# RWKV time mixing; norms around every sublayer)
+TINY_CONFIGS["W"] = {
+    "architecture": "Buzinex", "vocab": 384, "width": 128, "norm": {"eps": 1e-5}, "embedding": {"scale": 11.0}, "logit_scale": 0.7,
+    "logit_softcap": 25.0, "max_positions": 512,
+    "layers": [{"type": kind, "mixer": mixer, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+               for kind, mixer, ff in (
+                   ("wkv", {"heads": 2, "dim": 64, "rank": 24}, None),
+                   ("latent_attention", {"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 48, "kv_rank": 64, "scale": 0.15, "mask": {"size": 20},
+                                         "rot": {"base": 10000.0, "dims": 16}}, 192),
+                   ("attention", {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 64, "scale": 0.18, "softcap": 25.0,
+                                  "q_temp": {"coef": 0.2, "every": 16}}, 160),
+                   ("latent_attention", {"heads": 2, "dim": 48, "rot_dim": 32, "vdim": 64, "kv_rank": 96, "scale": 0.11, "mask": {"size": 9},
+                                         "rot": {"base": 500.0, "dims": 32}}, 224))]}
+
 def _table(rows: list[dict]) -> str:
     if not rows:
         return "  (no work)"
@@ -254,7 +269,7 @@ def main(argv=None) -> int:
         p.add_argument("--tiny", choices=sorted(TINY) + sorted(TINY_CONFIGS), help="instead of --model: a tiny random model (A: 2 layers, "
                        "hidden 64, 4/2 heads of 16, tied head; B: 3 layers, hidden 96, 3/1 heads of 32, untied head; T: a Tulipel "
                        "model of 4 latent-attention layers, width 128; L: a Letanex model of 3 layers, width 128; V: a Vuripel model of "
-                       "3 layers of which two run twice, width 128; Z: a Zevedra model of 3 layers of which two run twice, width 128), written with --seed")
+                       "3 layers of which two run twice, width 128; Z: a Zevedra model of 3 layers of which two run twice, width 128; W: a Buzinex model of 4 layers, width 128), written with --seed")
         p.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16")
         p.add_argument("--seed", type=int, default=0)
     rnd = sub.add_parser("random-model", help="write config.json and model.safetensors with random weights")
