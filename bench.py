@@ -702,6 +702,20 @@ def _median_us(call, repeats: int = 10) -> float:
     return statistics.median(times)
 
 
+def _captured_us(call, repeats: int = 20) -> float:
+    """Device time of ``call`` from a captured graph of ``repeats`` of them: what a decode step, which replays a graph, pays for
+    it (calls of a few launches cost the host more than the device)."""
+    import torch
+    for _ in range(3):
+        call()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for _ in range(repeats):
+            call()
+    return _median_us(graph.replay, repeats=3) / repeats
+
+
 def timed_latent_kernels(shape: str, tokens: int, batch: int, context: int, peak: dict) -> dict:
     """The new design's attention kernels alone beside the grouped-query kernels at equal heads and head size:
     one prompt of ``tokens`` tokens (FLOPs of the causal half against the measured bf16 rate) and ``batch`` decode
@@ -1684,6 +1698,204 @@ def timed_zevedra(args) -> dict:
     return result
 
 
+BUZINEX_SHAPES = {
+    "1b": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, lat_dim=64, rot_dim=64, lat_vdim=128, kv_rank=512, window=1024,
+               state_heads=16, state_dim=128, rank=64, ff=4096, vocab=32768),
+    "0.3b": dict(width=1024, heads=8, kv_heads=2, dim=128, vdim=128, lat_dim=64, rot_dim=64, lat_vdim=128, kv_rank=256, window=512,
+                 state_heads=8, state_dim=128, rank=32, ff=2048, vocab=32768),
+}
+
+
+def buzinex_folders(shape: str, layers: int):
+    """(Buzinex folder, Tulipel folder, Rarutar folder of equal size), random weights, written once.  Buzinex's layers in fours:
+    RWKV time mixing, latent attention over a window, attention with growing queries and capped scores, latent attention again;
+    all with the gated feed-forward.  Tulipel (latent attention) and Rarutar (recurrences, windows) beside it at the same
+    width, heads, latent, window and vocabulary."""
+    from sprout_lm_b200 import parse_config, write_random_model
+    z = BUZINEX_SHAPES[shape]
+    latent = ("latent_attention", {"heads": z["heads"], "dim": z["lat_dim"], "rot_dim": z["rot_dim"], "vdim": z["lat_vdim"], "kv_rank": z["kv_rank"],
+                                   "scale": (z["lat_dim"] + z["rot_dim"]) ** -0.5, "mask": {"size": z["window"]},
+                                   "rot": {"base": 500000.0, "dims": z["rot_dim"]}})
+    kinds = [("wkv", {"heads": z["state_heads"], "dim": z["state_dim"], "rank": z["rank"]}), latent,
+             ("attention", {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+                            "softcap": 30.0, "q_temp": {"coef": 0.1, "every": 8192}}), latent]
+    raw = {"architecture": "Buzinex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+           "logit_scale": 0.5, "logit_softcap": 30.0, "max_positions": 16384,
+           "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": {"kind": "dense", "ff": z["ff"]}} for i in range(layers)]}
+    folder = Path(tempfile.gettempdir()) / f"sprout_lm_b200_bench_{os.getuid()}_buzinex_{shape}_L{layers}"
+    if not (folder / "complete").exists():
+        print(f"[bench] writing random weights to {folder}", file=sys.stderr, flush=True)
+        write_random_model(folder, parse_config(raw), seed=0)
+        (folder / "complete").write_text("ok")
+    return folder, latent_folders(shape, layers)[0], rarutar_folders(shape, layers)[0]
+
+
+def timed_buzinex_kernels(shape: str, tokens: int, batch: int, context: int, peak: dict) -> dict:
+    """Buzinex's kernels alone beside the like kernels of the closest models at equal sizes, for one prompt of ``tokens`` tokens
+    and for ``batch`` single tokens with ``context`` keys held.  Latent attention over a window beside the same over everything
+    and capped attention beside the same without a cap (executed FLOPs of the visible keys against the measured bf16 rate; bytes
+    of the visible keys against the measured copy rate); the recurrence with a bonus beside the scan with a decay per channel
+    (operations against the CUDA cores' nominal rate; bytes against the copy rate); the recurrence's five projections in one launch
+    beside one product of as many features over one input; blends, append, norms and the small row kernels beside the plainer
+    forms of each (bytes against the copy rate).  Single tokens are timed from captured graphs, as decode steps run."""
+    import torch
+    from types import SimpleNamespace
+    from sprout_lm_b200 import kernels
+    from sprout_lm_b200.parts.linear import GroupedLinear, Linear
+    z = BUZINEX_SHAPES[shape]
+    page, width, heads, kv = 16, z["width"], z["heads"], z["kv_heads"]
+    g = torch.Generator(device="cuda").manual_seed(0)
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    out = {}
+
+    def rand(*shape_, scale=1.0, dtype=torch.bfloat16):
+        return (torch.randn(*shape_, device="cuda", generator=g) * scale).to(dtype)
+
+    def moved(name, us, mb, **more):
+        out[name] = {"us": round(us, 1), "mb": round(mb, 2), "gbs": round(mb / us * 1e3), "of_measured_copy": round(mb / us * 1e3 / peak["hbm_gbs"], 3),
+                     **more}
+
+    def pairs(name, us, flops):
+        tflops = flops / us / 1e6
+        out[name] = {"us": round(us, 1), "tflops": round(tflops, 1), "of_measured_bf16": round(tflops / peak["bf16_tflops"], 3)}
+    try:
+        top_mhz = float(subprocess.run(["nvidia-smi", "--query-gpu=clocks.max.sm", "--format=csv,noheader,nounits", "-i", "0"],
+                                       capture_output=True, text=True, timeout=20).stdout.split()[0])
+    except (OSError, ValueError, IndexError, subprocess.SubprocessError):
+        top_mhz = 1965.0
+    fp32_tflops = torch.cuda.get_device_properties(0).multi_processor_count * 128 * 2 * top_mhz / 1e6
+    out["fp32_cuda_core_tflops_nominal"] = round(fp32_tflops, 1)
+    for label, requests, new, held in (("prefill", 1, tokens, tokens), ("decode", batch, 1, context)):
+        n = requests * new
+
+        def timed(call, new=new):
+            return _median_us(call, repeats=3) if new > 1 else _captured_us(call)
+        pages = -(-held // page)
+        table = torch.full((requests, -(-pages // 64) * 64), -1, dtype=torch.int32, device="cuda")
+        table[:, :pages] = torch.randperm(requests * pages, device="cuda", generator=g).to(torch.int32).reshape(requests, pages)
+        ctx = SimpleNamespace(seq_of_token=torch.arange(requests, dtype=torch.int32, device="cuda").repeat_interleave(new),
+                              positions=(torch.arange(new, dtype=torch.int32, device="cuda") + (held - new)).repeat(requests),
+                              q_start=(torch.arange(requests + 1, dtype=torch.int32, device="cuda") * new),
+                              context_lens=torch.full((requests,), held, dtype=torch.int32, device="cuda"), max_q_len=new, max_context=held,
+                              planned_context=0, num_seqs=requests, num_tokens=n)
+        # latent attention
+        rank, row = z["kv_rank"], z["kv_rank"] + z["rot_dim"]
+        cache, q = rand(requests * pages + 1, 1, page, row, scale=0.3), rand(n, heads * row, scale=0.3)
+        o = torch.empty(n, heads * rank, dtype=torch.bfloat16, device="cuda")
+        view = SimpleNamespace(k=cache, v=None, block_table=table, page_tokens=page, write=False)
+        sink = torch.zeros(heads, device="cuda")
+        near = SimpleNamespace(**{**vars(ctx), "max_context": min(held, z["window"]), "context_lens": ctx.context_lens.clamp(max=z["window"])})
+        variants = [("latent_window", ctx, z["window"]), ("tulipel_latent", ctx, 0)]
+        if new == 1:
+            variants.append(("tulipel_latent_equal_keys", near, 0))              # contexts as long as the window
+        for name, at, window in variants:
+            us = timed(lambda: kernels.latent_attention(q, view, at, sink, o, heads, rank, 0.09, status, window=window))
+            size = window or at.max_context
+            if new > 1:
+                pairs(f"{name}_{label}", us, 2.0 * heads * (row + rank) * sum(min(p + 1, size) for p in range(new)))
+            else:
+                moved(f"{name}_{label}", us, requests * min(held, size) * row * 2 / 1e6)
+        del cache, q, o
+        # attention with capped scores; append with norms and growing queries
+        dim, vdim = z["dim"], z["vdim"]
+        k2, v2 = rand(requests * pages + 1, kv, page, dim), rand(requests * pages + 1, kv, page, vdim)
+        rows = rand(n, heads * dim + kv * (dim + vdim), scale=0.3)
+        o2 = torch.empty(n, heads * vdim, dtype=torch.bfloat16, device="cuda")
+        view = SimpleNamespace(k=k2, v=v2, block_table=table, page_tokens=page, write=False)
+        for name, cap in (("capped", 30.0), ("plain", 0.0)):
+            us = timed(lambda: kernels.multimap_attention(rows[:, :heads * dim], view, ctx, o2, heads, kv, 1, dim, vdim, dim ** -0.5, 0.0, 0.0, 1.0,
+                                                               status, softcap=cap))
+            if new > 1:
+                pairs(f"{name}_attention_{label}", us, heads * (dim + vdim) * float(new) * (new + 1))
+            else:
+                moved(f"{name}_attention_{label}", us, requests * held * kv * (dim + vdim) * 2 / 1e6)
+        qw, kw = torch.ones(dim, device="cuda"), torch.ones(dim, device="cuda")
+        mb = n * (heads * dim * 2 + kv * (dim + vdim) * 2) * 2 / 1e6
+        for name, growth in (("append_growth", (0.1, 512)), ("append_vuripel", None)):
+            us = timed(lambda: kernels.rope_maps_append(rows, ctx.positions, ctx.seq_of_token, table, None, None, k2, v2, heads, kv, 1, dim, vdim,
+                                                             page, True, status, q_weight=qw, k_weight=kw, weight_eps=1e-5, growth=growth))
+            moved(f"{name}_{label}", us, mb)
+        del k2, v2, rows, o2
+        # RWKV time mixing
+        sh, sd = z["state_heads"], z["state_dim"]
+        sw, slots = sh * sd, torch.arange(requests, dtype=torch.int32, device="cuda")
+        h, mu = rand(n, width), rand(5, width, scale=0.3, dtype=torch.float32)
+        blended = torch.empty(n, 5 * width, dtype=torch.bfloat16, device="cuda")
+        before = SimpleNamespace(buffer=torch.zeros(requests, width, device="cuda"), slots=slots)
+        moved(f"token_blend_{label}", timed(lambda: kernels.token_blend(h, mu, blended, ctx, before, status)),
+              (n * width * 12 + requests * width * 8) / 1e6)
+        conv_in, conv_out, taps = rand(n, 3 * width), rand(n, 3 * width), rand(3 * width, 4, dtype=torch.float32)
+        conv_state = SimpleNamespace(buffer=torch.zeros(requests, 3, 3 * width, device="cuda"), slots=slots)
+        moved(f"short_conv_{label}", timed(lambda: kernels.causal_conv(conv_in, taps, None, conv_out, ctx, conv_state, status)),
+              (n * width * 12 + requests * 3 * width * 3 * 8) / 1e6)
+        del conv_in, conv_out
+        weights = [rand(rows_, width, scale=0.02) for rows_ in (sw, sw, sw, sw, z["rank"])]
+        grouped, single = GroupedLinear(weights, status), Linear(rand(4 * sw + 256, width, scale=0.02), None, status)
+        w_mb, features = (4 * sw + z["rank"]) * width * 2 / 1e6, 4 * sw + z["rank"]
+        for name, call, cols in (("five_products", lambda: grouped.forward_float32(blended), features), ("one_product", lambda: single.forward_float32(h), 4 * sw + 256)):
+            us = timed(call)
+            pairs(f"{name}_{label}", us, 2.0 * n * width * cols)
+            out[f"{name}_{label}"]["of_measured_copy"] = round((w_mb + n * cols * 4 / 1e6) / us * 1e3 / peak["hbm_gbs"], 3)
+        del weights, grouped, single
+        state = SimpleNamespace(buffer=torch.zeros(requests, sh, sd, sd, device="cuda"), slots=slots)
+        o = torch.empty(n, sw, device="cuda")
+        zed, bias, bonus = rand(n, sw, dtype=torch.float32), torch.full((sw,), -3.0, device="cuda"), torch.ones(sw, device="cuda")
+        state_mb = 2 * requests * sh * sd * sd * 4 / 1e6
+        for name, dtype, ops, options in (("bonus_scan", torch.float32, 6, dict(bonus=bonus)), ("channel_decay_scan", torch.bfloat16, 6, dict(tau=16.0))):
+            r, k, v = (rand(n, sw, scale=0.5, dtype=dtype) for _ in range(3))
+            us = timed(lambda: kernels.gated_scan(r, k, v, zed, bias, ctx, state, o, sh, sh, sd, sd, status, **options))
+            moved(f"{name}_{label}", us, n * sw * (3 * r.element_size() + 8) / 1e6 + state_mb,
+                  of_nominal_fp32_cores=round(ops * float(n) * sw * sd / us / 1e6 / fp32_tflops, 3))
+        gain, gated, y = torch.ones(sw, device="cuda"), torch.empty(n, sw, dtype=torch.bfloat16, device="cuda"), rand(n, sw, dtype=torch.float32)
+        for name, gate in (("head_norm_gate32", rand(n, sw, dtype=torch.float32)), ("head_norm_gate16", rand(n, sw))):
+            moved(f"{name}_{label}", timed(lambda: kernels.gated_group_norm(y, gate, gain, gated, 1e-5, groups=sh)), n * sw * (6 + gate.element_size()) / 1e6)
+        low, inner = torch.empty(n, z["rank"], dtype=torch.bfloat16, device="cuda"), rand(n, z["rank"], dtype=torch.float32)
+        moved(f"tanh_{label}", timed(lambda: kernels.unit_act(inner, low, "tanh", gated=False)), n * z["rank"] * 6 / 1e6)
+        # norms around the sublayers, the head's scale and cap
+        x, y, gain = rand(n, width, dtype=torch.float32), rand(n, width, dtype=torch.float32), torch.ones(width, device="cuda")
+        for name, rms, clear in (("rms_norm_add_next", True, True), ("layernorm_add_next", False, False)):
+            us = timed(lambda: kernels.norm_add(y, gain, x, 1e-5, next_gain=gain, h=h, rms=rms, clear=clear))
+            moved(f"{name}_{label}", us, n * width * (18 if clear else 14) / 1e6)
+        logits = rand(min(n, 64), z["vocab"], dtype=torch.float32)
+        for name, factor in (("scaled_cap", 0.5), ("cap", 1.0)):
+            moved(f"{name}_{label}", timed(lambda: kernels.softcap(logits, 30.0, factor=factor)), logits.numel() * 8 / 1e6)
+    assert int(status.item()) == 0
+    return out
+
+
+def timed_buzinex(args) -> dict:
+    """``--only buzinex``: prefill and decode throughput of Buzinex at ``--shape 1b|0.3b`` (random weights, ``--layers`` layers,
+    4 if not given) beside Tulipel and Rarutar at equal size, through the same runner, and the kernels alone."""
+    import numpy as np
+    import torch
+    from sprout_lm_b200 import load_model
+    from sprout_lm_b200.engine.step import ModelRunner
+    shape = args.shape if args.shape in BUZINEX_SHAPES else "1b"
+    layers = args.layers or 4
+    peak = peaks()
+    folders = buzinex_folders(shape, layers)
+    prompt_len = args.prompt_len
+    result = {"impl": "ours", "only": "buzinex", "shape": shape, "layers": layers, "dtype": "bf16", "data": "synthetic",
+              "prefill_tokens": args.tokens, "decode_batch": args.batch, "decode_prompt_len": prompt_len, "steps": args.steps,
+              "peaks": {"bf16_tflops": peak["bf16_tflops"], "hbm_gbs": peak["hbm_gbs"], "source": peak.get("source", "measured")}}
+    for tag, folder in zip(("buzinex", "tulipel", "rarutar"), folders):
+        model = load_model(folder, dtype="bfloat16", device="cuda:0")
+        slots = max(64, args.batch)
+        pages = slots * (-(-(prompt_len + args.steps + args.warmup + 16) // 16)) + args.tokens // 16 + 16
+        runner = ModelRunner(model, num_pages=pages, page_tokens=16, max_requests=slots, prefix_caching=False)
+        rng = np.random.default_rng(0)
+        ms = timed_prefill(runner, args.tokens, rng)
+        decode = timed_decode(runner, args.batch, prompt_len, args.steps, args.warmup, rng)
+        result[tag] = {"weights_mb": round((folder / "model.safetensors").stat().st_size / 1e6, 1), "prefill_ms": round(ms, 3),
+                       "prefill_tokens_per_s": round(args.tokens / ms * 1000),
+                       "decode_ms_per_step": round(decode["ms_per_step"], 4), "decode_tokens_per_s": round(decode["tokens_per_s"]),
+                       "decode_launches_per_step": decode["launches_per_step"]}
+        del runner, model
+        torch.cuda.empty_cache()
+    result["kernels"] = timed_buzinex_kernels(shape, args.tokens, max(args.batch, 64), 2048, peak)
+    return result
+
+
 def run(args) -> dict:
     import numpy as np
     import torch
@@ -1701,6 +1913,8 @@ def run(args) -> dict:
         return timed_vuripel(args)
     if args.only == "zevedra":
         return timed_zevedra(args)
+    if args.only == "buzinex":
+        return timed_buzinex(args)
     if args.only == "attention":
         return timed_attention(args.tokens, args.shape)
     if args.only == "gemm":
@@ -1808,7 +2022,7 @@ def main() -> int:
     parser.add_argument("--portion", type=int, default=4096, help="with --only long-prompt: tokens of a step (--tokens: of the whole prompt)")
     parser.add_argument("--prompt-len", type=int, default=512, help="with --only decode: tokens of every request's prompt (the context grows to hold it)")
     parser.add_argument("--layers", type=int, default=0, help="fewer layers than the model has (named in config)")
-    parser.add_argument("--only", choices=["all", "decode", "prefill", "ablate", "attention", "decode-attention", "gemm", "serve", "long-prompt", "latent", "letanex", "rarutar", "vuripel", "zevedra"], default="all",
+    parser.add_argument("--only", choices=["all", "decode", "prefill", "ablate", "attention", "decode-attention", "gemm", "serve", "long-prompt", "latent", "letanex", "rarutar", "vuripel", "zevedra", "buzinex"], default="all",
                         help="measure one part only (for profiling captures); the JSON line then holds that part")
     parser.add_argument("--shape", choices=sorted(set(SHAPES) | set(LATENT_SHAPES) | set(LETANEX_SHAPES) | set(RARUTAR_SHAPES)), default="0.5b", help="with --only: the model's sizes")
     parser.add_argument("--requests", type=int, default=64, help="with --only serve: requests of the workload")

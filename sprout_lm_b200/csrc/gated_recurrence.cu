@@ -472,6 +472,16 @@ token_blend_kernel(const T* __restrict__ h, const float* __restrict__ mu, T* __r
         for (int i = 0; i < VEC; i++) v[i] = to_float(src[i]);
       }
     };
+    auto floats = [&](const float* src, float (&v)[VEC]) {
+      if (VEC == 8) {
+        const float4 a = reinterpret_cast<const float4*>(src)[0], b = reinterpret_cast<const float4*>(src)[1];
+        v[0] = a.x; v[1 % VEC] = a.y; v[2 % VEC] = a.z; v[3 % VEC] = a.w;
+        v[4 % VEC] = b.x; v[5 % VEC] = b.y; v[6 % VEC] = b.z; v[7 % VEC] = b.w;
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; i++) v[i] = src[i];
+      }
+    };
     row(t, now);
     if (t > begin) {
       row(t - 1, delta);
@@ -485,17 +495,22 @@ token_blend_kernel(const T* __restrict__ h, const float* __restrict__ mu, T* __r
         float* mine = state + (size_t)slot * width + c;
         float last[VEC];
         row(q_start[r + 1] - 1, last);
+        floats(mine, delta);
+        if (VEC == 8) {
+          reinterpret_cast<float4*>(mine)[0] = make_float4(last[0], last[1 % VEC], last[2 % VEC], last[3 % VEC]);
+          reinterpret_cast<float4*>(mine)[1] = make_float4(last[4 % VEC], last[5 % VEC], last[6 % VEC], last[7 % VEC]);
+        } else {
 #pragma unroll
-        for (int i = 0; i < VEC; i++) {
-          delta[i] = mine[i];
-          mine[i] = last[i];
+          for (int i = 0; i < VEC; i++) mine[i] = last[i];
         }
       }
     }
 #pragma unroll
     for (int i = 0; i < VEC; i++) delta[i] -= now[i];
+#pragma unroll 5
     for (int s = 0; s < parts; s++) {
-      const float* m = mu + (size_t)s * width + c;
+      float m[VEC];
+      floats(mu + (size_t)s * width + c, m);
       T* dst = out + ((size_t)t * parts + s) * width + c;
       if (VEC == 8 && sizeof(T) == 2) {
         uint4 packed;
@@ -673,17 +688,20 @@ SPROUT_API int sprout_token_blend(const void* h, const float* mu, void* out, int
                                   cudaStream_t stream) {
   SPROUT_REQUIRE(h && mu && out && q_start && seq_of_token && state_slots && state && status, "token_blend: null pointer");
   SPROUT_REQUIRE(tokens > 0 && width > 0 && parts > 0 && num_slots > 0, "token_blend: bad sizes");
-  const bool vec = dtype == SPROUT_BF16 && width % 8 == 0 && (((uintptr_t)h | (uintptr_t)out) & 15) == 0;
-  const long long blocks = ((long long)tokens * (width / (vec ? 8 : 1)) + 255) / 256;
+  const bool vec = dtype == SPROUT_BF16 && width % 8 == 0 && (((uintptr_t)h | (uintptr_t)out | (uintptr_t)mu | (uintptr_t)state) & 15) == 0;
+  // few tokens: small blocks, so that more SMs have one
+  const long long threads = (long long)tokens * (width / (vec ? 8 : 1));
+  const int block = threads < 148 * 256 ? 64 : 256;
+  const long long blocks = (threads + block - 1) / block;
   const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
   if (dtype == SPROUT_F32)
-    sprout_launch(token_blend_kernel<float, 1>, grid, dim3(256), 0, stream, (const float*)h, mu, (float*)out, q_start, seq_of_token,
+    sprout_launch(token_blend_kernel<float, 1>, grid, dim3(block), 0, stream, (const float*)h, mu, (float*)out, q_start, seq_of_token,
                   state_slots, state, num_slots, tokens, width, parts, status);
   else if (vec)
-    sprout_launch(token_blend_kernel<__nv_bfloat16, 8>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)h, mu, (__nv_bfloat16*)out,
+    sprout_launch(token_blend_kernel<__nv_bfloat16, 8>, grid, dim3(block), 0, stream, (const __nv_bfloat16*)h, mu, (__nv_bfloat16*)out,
                   q_start, seq_of_token, state_slots, state, num_slots, tokens, width, parts, status);
   else if (dtype == SPROUT_BF16)
-    sprout_launch(token_blend_kernel<__nv_bfloat16, 1>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)h, mu, (__nv_bfloat16*)out,
+    sprout_launch(token_blend_kernel<__nv_bfloat16, 1>, grid, dim3(block), 0, stream, (const __nv_bfloat16*)h, mu, (__nv_bfloat16*)out,
                   q_start, seq_of_token, state_slots, state, num_slots, tokens, width, parts, status);
   else
     return sprout_fail("token_blend: unknown dtype %d", dtype);
